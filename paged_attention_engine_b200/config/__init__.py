@@ -3,12 +3,13 @@ from .engine_config import EngineConfig
 from .errors import ConfigError
 from .bidonex import BidonexConfig
 from .finezen import FinezenConfig
+from .getozen import GetozenConfig
 from .qwen2 import Qwen2Config
 from .pukerax import PukeraxConfig
 from .zugarax import ZugaraxConfig
 from .registry import ARCHITECTURES, Architecture, register_architecture, resolve, resolve_folder
 
 __all__ = [
-    "ARCHITECTURES", "Architecture", "BidonexConfig", "ConfigError", "EngineConfig", "FinezenConfig", "LayerSpec", "ModelSpec", "PartSpec", "Qwen2Config",
+    "ARCHITECTURES", "Architecture", "BidonexConfig", "ConfigError", "EngineConfig", "FinezenConfig", "GetozenConfig", "LayerSpec", "ModelSpec", "PartSpec", "Qwen2Config",
     "PukeraxConfig", "ScheduleEntry", "ZugaraxConfig", "register_architecture", "resolve", "resolve_folder",
 ]

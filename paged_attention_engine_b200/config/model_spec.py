@@ -86,6 +86,8 @@ class ModelSpec:
     schedule: tuple[ScheduleEntry, ...]
     final_norm: PartSpec
     head: PartSpec
+    # tensors that a checkpoint of the architecture may hold although nothing reads them
+    unread: tuple[str, ...] = ()
 
     def __post_init__(self) -> None:
         for pos, entry in enumerate(self.schedule):

@@ -18,6 +18,7 @@ from .errors import ConfigError
 from .model_spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
 from .bidonex import BidonexConfig
 from .finezen import FinezenConfig
+from .getozen import GetozenConfig
 from .qwen2 import Qwen2Config
 from .pukerax import PukeraxConfig
 from .zugarax import ZugaraxConfig
@@ -451,3 +452,80 @@ def finezen_spec(cfg: FinezenConfig) -> ModelSpec:
 
 
 register_architecture("Finezen", FinezenConfig, finezen_spec)
+
+
+# --------------------------------------------------------------------------- #
+# Getozen: a token embedding into a float32 residual stream; each layer's two branches read the same
+# stream through a norm without statistics each, x <- x + mixer(dyt_1(x)) + ff(dyt_2(x)); the mixer an
+# attention (biased q, k and v, neighbouring channels rotated, linearly scaled frequencies, every
+# earlier key, a gate per channel) and a retention (fixed decay per head) side by side, their outputs
+# weighted by two constants, or the selective state space of Mamba-2; the feed-forward gated by a
+# rectifier, or absent; a layer may run with another's weights and a cache and state of its own;
+# the same norm and an untied head at the end.
+# --------------------------------------------------------------------------- #
+
+# The design has no longest sequence; positions are 32-bit integers.
+GETOZEN_MAX_POSITIONS = 1 << 30
+
+
+def getozen_spec(cfg: GetozenConfig) -> ModelSpec:
+    layers, place, unread = [], {}, []
+
+    def rotation(rot):
+        scaling = dict(rot.scaling, kind="linear") if rot.scaling is not None else None
+        return {"kind": "scaled_rotary", "dims": rot.dims, "base": rot.base, "scaling": scaling}
+
+    for i, layer in enumerate(cfg.layers):
+        if layer.weights_of is not None:
+            continue
+        prefix = f"l{i}"
+        m = layer.mixer
+        if layer.type == "parallel":
+            left = {
+                "hidden_size": cfg.width, "num_heads": m.left.heads, "num_kv_heads": m.left.kv_heads, "head_dim": m.left.dim,
+                "value_dim": m.left.vdim, "scale": m.left.scale, "window": 0, "qk_norm_eps": None, "qkv_bias": True,
+                "output_gate": True, "pairing": "interleaved", "position_encoding": rotation(m.left.rot),
+            }
+            right = {
+                "hidden_size": cfg.width, "num_heads": m.right.heads, "head_dim": m.right.dim, "value_dim": m.right.vdim,
+                "decay": m.right.decay, "norm_eps": cfg.norm_eps, "pairing": "half", "position_encoding": rotation(m.right.rot),
+            }
+            mixer = PartSpec("side_by_side", {"mixers": [
+                {"kind": "gated_window_attention", "params": left, "name": "left", "scale": m.left_scale},
+                {"kind": "retention", "params": right, "name": "right", "scale": m.right_scale}]}, f"{prefix}.mix")
+        else:
+            mixer = PartSpec(
+                "state_space",
+                {"hidden_size": cfg.width, "num_heads": m.heads, "value_dim": m.vdim, "state_dim": m.state, "groups": m.groups,
+                 "conv_taps": m.conv, "norm_groups": m.norm_groups, "norm_eps": cfg.norm_eps},
+                f"{prefix}.mix",
+            )
+        norm = lambda name: PartSpec("dynamic_tanh", {"size": cfg.width},
+                                     names={"weight": f"{prefix}.{name}", "alpha": f"{prefix}.{name}.alpha", "bias": f"{prefix}.{name}.b"})
+        place[i] = len(layers)
+        if layer.ff:
+            layers.append(LayerSpec("parallel_two_norms", dict(
+                mixer_norm=norm("norm1"), mixer=mixer, feed_forward_norm=norm("norm2"),
+                feed_forward=PartSpec("gated_mlp", {"hidden_size": cfg.width, "intermediate_size": layer.ff, "activation": "relu"},
+                                      f"{prefix}.mlp"))))
+        else:
+            # the branch that is absent may still have its norm in the checkpoint
+            unread += [f"{prefix}.norm2", f"{prefix}.norm2.alpha", f"{prefix}.norm2.b"]
+            layers.append(LayerSpec("summed_mixer", dict(norm=norm("norm1"), mixer=mixer)))
+    return ModelSpec(
+        architecture=cfg.architecture,
+        vocab_size=cfg.vocab,
+        hidden_size=cfg.width,
+        max_positions=GETOZEN_MAX_POSITIONS,
+        embedding=PartSpec("scaled_token_embedding", {"vocab_size": cfg.vocab, "hidden_size": cfg.width, "scale": 1.0},
+                           names={"weight": "embed"}),
+        layers=tuple(layers),
+        schedule=tuple(ScheduleEntry(place[i if layer.weights_of is None else layer.weights_of]) for i, layer in enumerate(cfg.layers)),
+        final_norm=PartSpec("dynamic_tanh", {"size": cfg.width},
+                            names={"weight": "final.norm", "alpha": "final.norm.alpha", "bias": "final.norm.b"}),
+        head=PartSpec("lm_head", {"vocab_size": cfg.vocab, "hidden_size": cfg.width, "tied_to": None}, names={"weight": "head"}),
+        unread=tuple(unread),
+    )
+
+
+register_architecture("Getozen", GetozenConfig, getozen_spec)

@@ -115,6 +115,13 @@ __device__ __forceinline__ int checked_page(int page) {
   return page;
 }
 
+// The gate of a gated linear unit, act(g) * u: SiLU, or the rectifier. The kernels that fold it
+// into a product's epilogue and the ones that run it alone all call this.
+enum GateKind : int { kGateSilu = 0, kGateRelu = 1 };
+__device__ __forceinline__ float gated(float g, float u, int kind) {
+  return kind == kGateRelu ? fmaxf(g, 0.f) * u : g / (1.f + expf(-g)) * u;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

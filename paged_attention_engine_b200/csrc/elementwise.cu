@@ -295,11 +295,11 @@ PAE_EXPORT int pae_rotary_qk_cache_write(void* qkv, const float* table, const in
 }
 
 // ------------------------------------------------------------------------------------
-// SwiGLU's middle (engine/model.py:317-320): out[t, i] = silu(gate[t, i]) * up[t, i]
+// The middle of a gated feed-forward (engine/model.py:317-320): out[t, i] = act(gate[t, i]) * up[t, i], SiLU or the rectifier,
 // where a row of the input holds the gate in [0, I) and the up projection in [I, 2I).
 // ------------------------------------------------------------------------------------
 template <typename T>
-__global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gate_up, long long total, int inter, int block) {
+__global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gate_up, long long total, int inter, int block, int gate_kind) {
   dependent_launch_prologue();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total) return;
@@ -310,12 +310,12 @@ __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gate_
   const int up_col = block > 0 ? gate_col + block : inter + c;
   const float g = to_float(gate_up[t * 2 * inter + gate_col]);
   const float u = to_float(gate_up[t * 2 * inter + up_col]);
-  out[i] = from_float<T>(g / (1.f + expf(-g)) * u);
+  out[i] = from_float<T>(gated(g, u, gate_kind));
 }
 
 // bfloat16 rows whose half-width is a multiple of 8: eight columns per thread, 16-byte accesses.
 __global__ void silu_mul_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gate_up,
-                                       long long total_chunks, int inter) {
+                                       long long total_chunks, int inter, int gate_kind) {
   dependent_launch_prologue();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total_chunks) return;
@@ -331,26 +331,26 @@ __global__ void silu_mul_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
     const float2 gf = __bfloat1622float2(g[e]), uf = __bfloat1622float2(u[e]);
-    o[e] = __floats2bfloat162_rn(gf.x / (1.f + expf(-gf.x)) * uf.x, gf.y / (1.f + expf(-gf.y)) * uf.y);
+    o[e] = __floats2bfloat162_rn(gated(gf.x, uf.x, gate_kind), gated(gf.y, uf.y, gate_kind));
   }
   *(uint4*)(out + t * inter + c * 8) = packed;
 }
 
-PAE_EXPORT int pae_silu_mul(void* out, const void* gate_up, int tokens, int inter, int block, int dtype, void* stream) {
+PAE_EXPORT int pae_silu_mul(void* out, const void* gate_up, int tokens, int inter, int block, int gate_kind, int dtype, void* stream) {
   const long long n = (long long)tokens * inter;
   if (n == 0) return 0;
   if (block == 0 && dtype == kBF16 && inter % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0) {
     const long long chunks = n / 8;
     launch_kernel(silu_mul_bf16x8_kernel, (unsigned)((chunks + 255) / 256), 256, 0, (cudaStream_t)stream, 
-        (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, chunks, inter);
+        (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, chunks, inter, gate_kind);
     return check_launch("silu_mul");
   }
   const unsigned blocks = (unsigned)((n + 255) / 256);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == kF32)
-    launch_kernel(silu_mul_kernel<float>, blocks, 256, 0, s, (float*)out, (const float*)gate_up, n, inter, block);
+    launch_kernel(silu_mul_kernel<float>, blocks, 256, 0, s, (float*)out, (const float*)gate_up, n, inter, block, gate_kind);
   else if (dtype == kBF16)
-    launch_kernel(silu_mul_kernel<__nv_bfloat16>, blocks, 256, 0, s, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, n, inter, block);
+    launch_kernel(silu_mul_kernel<__nv_bfloat16>, blocks, 256, 0, s, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, n, inter, block, gate_kind);
   else
     return fail(1, "silu_mul: unknown dtype %d", dtype);
   return check_launch("silu_mul");

@@ -191,10 +191,10 @@ __global__ void __launch_bounds__(512) splitk_rms_norm_x4_kernel(T* __restrict__
     normed[(size_t)row * width + i] = from_float<T>(row_values[i] * scale * weight[i]);
 }
 
-// out[t, i] = silu(g) * u with g, u the rounded sums of columns i and inter + i.
+// out[t, i] = act(g) * u (SiLU or the rectifier) with g, u the rounded sums of columns i and inter + i.
 template <typename T>
 __global__ void splitk_silu_mul_kernel(T* __restrict__ out, const float* __restrict__ partial, int splits, int tokens,
-                                       int inter, int block) {
+                                       int inter, int block, int gate_kind) {
   dependent_launch_prologue();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (long long)tokens * inter) return;
@@ -206,7 +206,7 @@ __global__ void splitk_silu_mul_kernel(T* __restrict__ out, const float* __restr
   const int up_col = block > 0 ? gate_col + block : inter + c;
   const float g = to_float(from_float<T>(split_sum(partial, splits, plane, (size_t)t * 2 * inter + gate_col)));
   const float u = to_float(from_float<T>(split_sum(partial, splits, plane, (size_t)t * 2 * inter + up_col)));
-  out[i] = from_float<T>(g / (1.f + expf(-g)) * u);
+  out[i] = from_float<T>(gated(g, u, gate_kind));
 }
 
 // qkv[t, head, :] = round(sum + bias), q and k rotated, k and v written to their pages
@@ -462,16 +462,16 @@ PAE_EXPORT int pae_splitk_rms_norm(void* normed, void* value, const float* parti
   return check_launch("splitk_rms_norm");
 }
 
-PAE_EXPORT int pae_splitk_silu_mul(void* out, const float* partial, int splits, int tokens, int inter, int block,
+PAE_EXPORT int pae_splitk_silu_mul(void* out, const float* partial, int splits, int tokens, int inter, int block, int gate_kind,
                                    int dtype, void* stream) {
   const long long n = (long long)tokens * inter;
   if (n == 0) return 0;
   const unsigned blocks = (unsigned)((n + 255) / 256);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == kBF16)
-    launch_kernel(splitk_silu_mul_kernel<__nv_bfloat16>, blocks, 256, 0, s, (__nv_bfloat16*)out, partial, splits, tokens, inter, block);
+    launch_kernel(splitk_silu_mul_kernel<__nv_bfloat16>, blocks, 256, 0, s, (__nv_bfloat16*)out, partial, splits, tokens, inter, block, gate_kind);
   else if (dtype == kF32)
-    launch_kernel(splitk_silu_mul_kernel<float>, blocks, 256, 0, s, (float*)out, partial, splits, tokens, inter, block);
+    launch_kernel(splitk_silu_mul_kernel<float>, blocks, 256, 0, s, (float*)out, partial, splits, tokens, inter, block, gate_kind);
   else
     return fail(1, "splitk_silu_mul: unknown dtype %d", dtype);
   return check_launch("splitk_silu_mul");

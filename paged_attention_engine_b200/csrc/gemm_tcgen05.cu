@@ -49,7 +49,8 @@ struct Params {
   int planes;        // persistent kernel: K ranges per output tile, each summed into a float32 plane of its own (0 or 1: none)
   int ld_out;        // NORMAL: row pitch of out/residual in elements; SWAPPED: weight rows N
   int out_f32;
-  int swiglu;        // NORMAL only: columns come in blocks of 16 gate, 16 up; out[row, n / 2] = silu(gate) * up
+  int swiglu;        // NORMAL only: columns come in blocks of 16 gate, 16 up; out[row, n / 2] = act(gate) * up
+  int gate_kind;     // with swiglu: SiLU or the rectifier
   int activation;    // 0: none; 1: exact GELU, 2: tanh GELU, 3: squared ReLU, of the product (+ bias) rounded to the output's type, before the residual
   // q|k|v with rotation and page write in the epilogue (NORMAL, many tokens): out is
   // qkv [tokens, (heads + 2 kv_heads) d]; a tile of 256 columns holds whole heads.
@@ -169,7 +170,7 @@ __device__ __forceinline__ void store_row_chunk(const Params& p, int row, int co
     }
 }
 
-// SwiGLU in the epilogue: 16 gate columns and the 16 up columns that follow them give 16
+// A gated linear unit in the epilogue: 16 gate columns and the 16 up columns that follow them give 16
 // outputs. Gate and up are rounded to bfloat16 first, as the unfused path stores them.
 __device__ __forceinline__ void store_swiglu_chunk(const Params& p, int row, int col0, const float* g, const float* u) {
   __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)row * p.ld_out + (col0 >> 1);
@@ -181,7 +182,7 @@ __device__ __forceinline__ void store_swiglu_chunk(const Params& p, int row, int
   for (int i = 0; i < 16; ++i) {
     const float gg = __bfloat162float(__float2bfloat16_rn(g[i]));
     const float uu = __bfloat162float(__float2bfloat16_rn(u[i]));
-    r[i] = gg / (1.f + expf(-gg)) * uu;
+    r[i] = gated(gg, uu, p.gate_kind);
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -793,11 +794,11 @@ int check_operands(const void* x, const void* w, int k) {
 
 // out[tokens, n] = x[tokens, k] . w[n, k]^T (+ bias[n]) (+ residual[tokens, n]); x, w, residual
 // bfloat16, bias float32, out bfloat16 or float32 (then residual is float32 too).
-// out[tokens, n / 2] = silu(gate) * up where x . w^T gives gate and up in alternating blocks of 16
+// out[tokens, n / 2] = act(gate) * up (gate_kind 0: SiLU, 1: the rectifier) where x . w^T gives gate and up in alternating blocks of 16
 // columns (w's rows are laid out that way); many tokens only (the persistent kernel). n is a
 // multiple of 32 and at least 256.
-PAE_EXPORT int pae_linear_swiglu_tcgen05(void* out, const void* x, const void* w, int tokens, int n, int k, int* error,
-                                         void* stream) {
+PAE_EXPORT int pae_linear_swiglu_tcgen05(void* out, const void* x, const void* w, int tokens, int n, int k, int gate_kind,
+                                         int* error, void* stream) {
   if (tokens == 0 || n == 0) return 0;
   if (n % 32 || n < 256) return fail(2, "linear_swiglu_tcgen05: %d columns are not a multiple of 32 of at least 256", n);
   if (int err = check_operands(x, w, k)) return err;
@@ -809,6 +810,7 @@ PAE_EXPORT int pae_linear_swiglu_tcgen05(void* out, const void* x, const void* w
   p.kb_per_split = p.k_blocks;
   p.ld_out = n / 2;
   p.swiglu = 1;
+  p.gate_kind = gate_kind;
   p.error = error;
   return launch_persistent(p, x, w, k, (cudaStream_t)stream);
 }

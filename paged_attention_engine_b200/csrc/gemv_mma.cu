@@ -16,7 +16,7 @@
 //             the token (the product runs over x * norm weight; rsqrt(mean x^2 + eps) is one
 //             factor per token and is applied to the sums), bias, rounding, rotation, page write.
 //   gate|up   8 gate rows and their 8 up rows (the weight's rows alternate in blocks of 16):
-//             epilogue = scale, rounding, SiLU(gate) * up.
+//             epilogue = scale, rounding, act(gate) * up (SiLU or the rectifier).
 //   o, down   16 neighbouring rows; epilogue = + residual, rounding.
 //
 // Weights: every warp runs a ring of its own, filled by TMA and watched through one mbarrier
@@ -95,6 +95,7 @@ struct Params {
   // RESIDUAL
   const __nv_bfloat16* residual; // [tokens, n] or null
   __nv_bfloat16* out;            // RESIDUAL: [tokens, n]; GATE_UP: [tokens, n / 2]; QKV: [tokens, n]
+  int gate_kind;                 // GATE_UP: SiLU or the rectifier
   // QKV
   const float* bias;             // [n] or null
   const float* rotary;           // [tokens, d]: cosines then sines, or null
@@ -441,7 +442,7 @@ __global__ void __launch_bounds__(WARPS * 32) gemv_kernel(const __grid_constant_
       } else if (KIND == GATE_UP) {
         const int j = tile * 8 + g;
         const float gate = __bfloat162float(__float2bfloat16_rn(lo)), up = __bfloat162float(__float2bfloat16_rn(hi));
-        p.out[(size_t)token * (p.n >> 1) + j] = __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+        p.out[(size_t)token * (p.n >> 1) + j] = __float2bfloat16_rn(gated(gate, up, p.gate_kind));
       } else {
         const int row_lo = tile * ROWS + g, row_hi = row_lo + 8;
         if (row_lo < p.n) {
@@ -695,10 +696,10 @@ PAE_EXPORT int pae_linear_few_tokens(void* out, const void* x, const void* w, co
   return launch_tokens<RESIDUAL, true>(p, w, (n + ROWS - 1) / ROWS, (cudaStream_t)stream);
 }
 
-// out[token, inter] = SiLU(g) * u with g, u = RMSNorm(x) . (gate, up rows of w)^T, each rounded to
+// out[token, inter] = act(g) * u (gate_kind 0: SiLU, 1: the rectifier) with g, u = RMSNorm(x) . (gate, up rows of w)^T, each rounded to
 // bfloat16 first; w [2 inter, k] with rows alternating in blocks of 16 gate, 16 up.
 PAE_EXPORT int pae_linear_swiglu_few_tokens(void* out, const void* x, const void* w, const float* norm_weight, float eps,
-                                            int tokens, int two_inter, int k, int* error, void* stream) {
+                                            int tokens, int two_inter, int k, int gate_kind, int* error, void* stream) {
   if (int err = check_common("linear_swiglu_few_tokens", w, x, norm_weight, error, tokens, two_inter, k)) return err;
   if (two_inter % 32) return fail(2, "linear_swiglu_few_tokens: %d rows are not blocks of 16 gate and 16 up rows", two_inter);
   Params p{};
@@ -709,6 +710,7 @@ PAE_EXPORT int pae_linear_swiglu_few_tokens(void* out, const void* x, const void
   p.norm_weight = norm_weight;
   p.eps = eps;
   p.out = (__nv_bfloat16*)out;
+  p.gate_kind = gate_kind;
   p.error = error;
   return launch_tokens<GATE_UP, false>(p, w, two_inter / 16, (cudaStream_t)stream);
 }

@@ -27,18 +27,19 @@ namespace {
 
 struct HeadPrep {
   const void* proj;      // [tokens, ld]
-  void* q_out;           // [tokens, heads, qd]
+  void* q_out;           // [tokens, heads, qd], a row every q_ld elements
   void* keys;            // [pages, kv_heads, page_size, kd]
   void* values;          // [pages, kv_heads, page_size, dv]
   const float* q_norm;   // [q_span] or null
   const float* k_norm;   // [k_span] or null
   const float* table;    // [tokens, dims]: cosines, then sines; null: no rotation
-  const int* slots;      // [tokens]: page * page_size + offset, negative: nothing is written; null: no pages
-  int ld, q_off, k_off, v_off;
+  const int* slots;      // [tokens]: page * page_size + offset, negative: nothing is written; null: no pages (or `direct`)
+  int ld, q_ld, q_off, k_off, v_off;
   int heads, kv_heads, qd, kd, dv;
   int q_span, k_span, q_rot0, k_rot0, dims, interleaved, page_size;
   float eps;
   int whole;             // the norm's mean runs over all query (key) heads of the token; weights [heads, span]
+  int direct;            // keys and values leave as plain rows [tokens, kv_heads, d], as the queries do
   int whole_kv_heads;    // the key heads that the mean runs over (kv_heads is 0 in a step that writes no page)
 };
 
@@ -59,6 +60,7 @@ __global__ void __launch_bounds__(WARPS * 32) head_prep_kernel(const HeadPrep p)
     slot = p.slots[t];
     if (slot >= 0 && !slot_in_pool(slot, p.page_size)) slot = -1;
   }
+  if (p.direct) slot = t;                      // a page of one token each
   const int page = slot >= 0 ? slot / p.page_size : 0, offset = slot >= 0 ? slot - page * p.page_size : 0;
   const int half = p.dims >> 1;
   // "whole": the token's two sums of squares, by the whole block in an order that depends on
@@ -128,7 +130,7 @@ __global__ void __launch_bounds__(WARPS * 32) head_prep_kernel(const HeadPrep p)
     }
     TO* to;
     if (is_q)
-      to = (TO*)p.q_out + ((size_t)t * p.heads + index) * d;
+      to = (TO*)p.q_out + (size_t)t * p.q_ld + (size_t)index * d;
     else
       to = (TO*)(is_k ? p.keys : p.values) + (((size_t)page * p.kv_heads + index) * p.page_size + offset) * d;
     for (int i = lane; i < d; i += 32) to[i] = from_float<TO>(buf[i]);
@@ -151,41 +153,67 @@ __global__ void rotary_table_amplitude_kernel(float* __restrict__ table, const i
   table[(size_t)t * 2 * half + half + f] = s * amplitude;
 }
 
-// out[t, c] = x[t, c] * sigmoid(gate[t, gate_off + c / group]); the gate is a column range of a
-// projection, one column for every `group` neighbouring channels (a head's size: a gate per head).
+// out[t, out_off + c] = mult * x[t, c] * sigmoid(gate[t, gate_off + c / group]); the gate is a column
+// range of a projection, one column for every `group` neighbouring channels (a head's size: a gate
+// per head); the result is a column range of rows of out_ld elements.
+struct GateOut {
+  int width, out_ld, out_off, gate_ld, gate_off, group;
+  float mult;
+};
+
 template <typename TX, typename TG>
-__global__ void sigmoid_gate_kernel(TX* __restrict__ out, const TX* __restrict__ x, const TG* __restrict__ gate,
-                                    long long total, int width, int gate_ld, int gate_off, int group) {
+__global__ void sigmoid_gate_kernel(TX* __restrict__ out, const TX* __restrict__ x, const TG* __restrict__ gate, long long total,
+                                    const GateOut p) {
   dependent_launch_prologue();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total) return;
-  const long long t = i / width;
-  const int c = (int)(i - t * width);
-  const float g = to_float(gate[t * gate_ld + gate_off + c / group]);
-  out[i] = from_float<TX>(to_float(x[i]) / (1.f + expf(-g)));
+  const long long t = i / p.width;
+  const int c = (int)(i - t * p.width);
+  const float g = to_float(gate[t * p.gate_ld + p.gate_off + c / p.group]);
+  out[t * p.out_ld + p.out_off + c] = from_float<TX>(p.mult * to_float(x[i]) / (1.f + expf(-g)));
+}
+
+// The same for bfloat16 x, a float32 gate per channel and everything aligned: four channels a thread.
+__global__ void __launch_bounds__(256) sigmoid_gate4_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x,
+                                                            const float* __restrict__ gate, long long quads, const GateOut p) {
+  dependent_launch_prologue();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= quads) return;
+  const int per_row = p.width >> 2;
+  const long long t = i / per_row;
+  const int c = (int)(i - t * per_row) * 4;
+  const uint2 x4 = *(const uint2*)(x + t * p.width + c);
+  const float4 g4 = *(const float4*)(gate + t * p.gate_ld + p.gate_off + c);
+  const float2 lo = __bfloat1622float2(*(const __nv_bfloat162*)&x4.x), hi = __bfloat1622float2(*(const __nv_bfloat162*)&x4.y);
+  uint2 packed;
+  *(__nv_bfloat162*)&packed.x = __floats2bfloat162_rn(p.mult * lo.x / (1.f + expf(-g4.x)), p.mult * lo.y / (1.f + expf(-g4.y)));
+  *(__nv_bfloat162*)&packed.y = __floats2bfloat162_rn(p.mult * hi.x / (1.f + expf(-g4.z)), p.mult * hi.y / (1.f + expf(-g4.w)));
+  *(uint2*)(out + t * p.out_ld + p.out_off + c) = packed;
 }
 
 }  // namespace
 
+// direct: keys and values go to plain rows [tokens, kv_heads, d] instead of pages.
 // whole: the norms' means run over all heads at once (weights [heads * span]). in_dtype: the projection's element type; out_dtype: that of q_out and of the pages (0 float32, 1 bfloat16).
-PAE_EXPORT int pae_head_prep(void* q_out, void* keys, void* values, const void* proj, int ld, int q_off, int k_off,
+PAE_EXPORT int pae_head_prep(void* q_out, int q_ld, void* keys, void* values, const void* proj, int ld, int q_off, int k_off,
                              int v_off, int tokens, int heads, int kv_heads, int qd, int kd, int dv,
                              const float* q_norm, int q_span, const float* k_norm, int k_span, float eps,
                              const float* table, int dims, int interleaved, int q_rot0, int k_rot0, const int* slots,
-                             int page_size, int whole, int in_dtype, int out_dtype, void* stream) {
+                             int page_size, int whole, int direct, int in_dtype, int out_dtype, void* stream) {
   if (tokens == 0 || heads + kv_heads == 0) return 0;
   if (heads < 0 || kv_heads < 0 || qd < 0 || kd < 0 || dv < 0) return fail(2, "head_prep: a negative size");
   if (dims % 2) return fail(2, "head_prep: %d rotated channels are not pairs", dims);
   if (table != nullptr && ((heads > 0 && q_rot0 + dims > qd) || (kv_heads > 0 && k_rot0 + dims > kd)))
     return fail(2, "head_prep: %d rotated channels from %d and %d do not fit heads of %d and %d", dims, q_rot0, k_rot0, qd, kd);
   if (q_span > qd || k_span > kd) return fail(2, "head_prep: a norm over %d or %d channels of heads of %d and %d", q_span, k_span, qd, kd);
-  if (kv_heads > 0 && slots != nullptr && (keys == nullptr || page_size < 1)) return fail(2, "head_prep: slots without pages");
+  if (kv_heads > 0 && (slots != nullptr || direct) && (keys == nullptr || (page_size < 1 && !direct))) return fail(2, "head_prep: slots without pages");
   if (heads > 0 && q_out == nullptr) return fail(2, "head_prep: query heads without an output");
+  if (heads > 0 && q_ld < heads * qd) return fail(2, "head_prep: query rows of %d for %d heads of %d", q_ld, heads, qd);
   if (whole && ((q_norm != nullptr && q_span != qd) || (k_norm != nullptr && k_span != kd)))
     return fail(2, "head_prep: a norm over the whole projection covers every channel (%d of %d, %d of %d)", q_span, qd, k_span, kd);
-  HeadPrep p{proj, q_out, keys, values, q_norm, k_norm, table, slots, ld, q_off, k_off, v_off, heads,
-             slots != nullptr ? kv_heads : 0, qd, kd, dv, q_span, k_span, q_rot0, k_rot0, table != nullptr ? dims : 0,
-             interleaved, page_size < 1 ? 1 : page_size, eps, whole, kv_heads};
+  HeadPrep p{proj, q_out, keys, values, q_norm, k_norm, table, slots, ld, q_ld, q_off, k_off, v_off, heads,
+             slots != nullptr || direct ? kv_heads : 0, qd, kd, dv, q_span, k_span, q_rot0, k_rot0, table != nullptr ? dims : 0,
+             interleaved, direct || page_size < 1 ? 1 : page_size, eps, whole, direct, kv_heads};
   const int widest = qd > kd ? (qd > dv ? qd : dv) : (kd > dv ? kd : dv);
   const size_t smem = sizeof(float) * WARPS * (size_t)widest;
   if (smem > 48 * 1024) return fail(2, "head_prep: heads of %d channels are too wide", widest);
@@ -211,20 +239,27 @@ PAE_EXPORT int pae_rotary_table_amplitude(float* table, const int* positions, co
   return check_launch("rotary_table_amplitude");
 }
 
-// x, out [tokens, width] in x_dtype; gate [tokens, gate_ld] in gate_dtype, columns gate_off .. gate_off + width / group.
-PAE_EXPORT int pae_sigmoid_gate(void* out, const void* x, const void* gate, int tokens, int width, int gate_ld,
-                                int gate_off, int group, int x_dtype, int gate_dtype, void* stream) {
+// x [tokens, width] and out [tokens, out_ld] (columns out_off .. out_off + width) in x_dtype; gate [tokens,
+// gate_ld] in gate_dtype, columns gate_off .. gate_off + width / group.
+PAE_EXPORT int pae_sigmoid_gate(void* out, int out_ld, int out_off, const void* x, const void* gate, int tokens, int width,
+                                int gate_ld, int gate_off, int group, float mult, int x_dtype, int gate_dtype, void* stream) {
   const long long total = (long long)tokens * width;
   if (total == 0) return 0;
   if (group < 1 || width % group) return fail(2, "sigmoid_gate: rows of %d channels in groups of %d", width, group);
   if (gate_off < 0 || gate_off + width / group > gate_ld) return fail(2, "sigmoid_gate: columns %d..%d of rows of %d", gate_off, gate_off + width / group, gate_ld);
+  if (out_off < 0 || out_off + width > out_ld) return fail(2, "sigmoid_gate: output columns %d..%d of rows of %d", out_off, out_off + width, out_ld);
+  const GateOut p{width, out_ld, out_off, gate_ld, gate_off, group, mult};
   cudaStream_t s = (cudaStream_t)stream;
   using bf = __nv_bfloat16;
   const unsigned blocks = (unsigned)((total + 255) / 256);
   const int key = x_dtype * 10 + gate_dtype;
-  if (key == 0) launch_kernel(sigmoid_gate_kernel<float, float>, blocks, 256, 0, s, (float*)out, (const float*)x, (const float*)gate, total, width, gate_ld, gate_off, group);
-  else if (key == 10) launch_kernel(sigmoid_gate_kernel<bf, float>, blocks, 256, 0, s, (bf*)out, (const bf*)x, (const float*)gate, total, width, gate_ld, gate_off, group);
-  else if (key == 11) launch_kernel(sigmoid_gate_kernel<bf, bf>, blocks, 256, 0, s, (bf*)out, (const bf*)x, (const bf*)gate, total, width, gate_ld, gate_off, group);
+  if (key == 10 && group == 1 && ((width | out_ld | out_off | gate_ld | gate_off) & 3) == 0 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)gate) & 15) == 0) {
+    launch_kernel(sigmoid_gate4_kernel, (unsigned)((total / 4 + 255) / 256), 256, 0, s, (bf*)out, (const bf*)x, (const float*)gate, total / 4, p);
+    return check_launch("sigmoid_gate");
+  }
+  if (key == 0) launch_kernel(sigmoid_gate_kernel<float, float>, blocks, 256, 0, s, (float*)out, (const float*)x, (const float*)gate, total, p);
+  else if (key == 10) launch_kernel(sigmoid_gate_kernel<bf, float>, blocks, 256, 0, s, (bf*)out, (const bf*)x, (const float*)gate, total, p);
+  else if (key == 11) launch_kernel(sigmoid_gate_kernel<bf, bf>, blocks, 256, 0, s, (bf*)out, (const bf*)x, (const bf*)gate, total, p);
   else return fail(1, "sigmoid_gate: element types x=%d gate=%d are not supported", x_dtype, gate_dtype);
   return check_launch("sigmoid_gate");
 }

@@ -226,14 +226,15 @@ class PendingStreams:
 
 
 class PendingResidual:
-    """A float32 residual stream x + mult * post(y) (+ extra) whose sum has not been made: `residual_add`
+    """A float32 residual stream x + mult * post(y) (+ y2) (+ extra) whose sum has not been made: `residual_add`
     returns one, and the norm without statistics that reads the stream next (`dyt_norm`) makes the
     sum inside its own kernel; anything else calls `materialized`, which runs the sum alone. `post`
     is (alpha, weight, bias) of a Dynamic Tanh applied to y first, or None; y may be a product that is
-    still in its splits; `extra` is a second stream that joins (or None)."""
+    still in its splits; `y2` is the output of a second sublayer that ran beside the first (likewise, or
+    None); `extra` is a second stream that joins (or None)."""
 
-    def __init__(self, x, y, post, mult: float, extra=None) -> None:
-        self.x, self.y, self.post, self.mult, self.extra = x, y, post, float(mult), extra
+    def __init__(self, x, y, post, mult: float, extra=None, y2=None) -> None:
+        self.x, self.y, self.post, self.mult, self.extra, self.y2 = x, y, post, float(mult), extra, y2
         self.dtype = torch.float32
         self.value = None
 
@@ -794,8 +795,12 @@ def paged_attention(qkv, keys, values, block_table, q_start, q_pos0, kv_len, num
     return out
 
 
-def silu_mul(gate_up, block: int = 0) -> torch.Tensor:
-    """silu(gate) * up of a [tokens, 2 I] product. block 0: gate is columns [0, I) and up [I, 2 I);
+# The activations of a gated linear unit's gate.
+GATE_KINDS = {"silu": 0, "relu": 1}
+
+
+def silu_mul(gate_up, block: int = 0, gate: str = "silu") -> torch.Tensor:
+    """act(gate) * up (`gate`: "silu" or "relu") of a [tokens, 2 I] product. block 0: gate is columns [0, I) and up [I, 2 I);
     block b: b gate columns, then their b up columns, and so on (`linear_swiglu`'s weight layout)."""
     tokens, two_i = gate_up.shape
     if two_i % 2 or (block and two_i % (2 * block)):
@@ -806,13 +811,13 @@ def silu_mul(gate_up, block: int = 0) -> torch.Tensor:
         out = torch.empty((tokens, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
         lib = _lib("fused_decode")
         _check(lib, lib.pae_splitk_silu_mul(_ptr(out), _ptr(gate_up.partial), splits, tokens,
-                                            (two_i // 2), block, _DTYPE_CODE[gate_up.dtype], _stream()))
+                                            (two_i // 2), block, GATE_KINDS[gate], _DTYPE_CODE[gate_up.dtype], _stream()))
         return out
     gate_up = materialized(gate_up)
     _need(gate_up, "silu_mul: gate_up")
     out = torch.empty((tokens, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
     lib = _lib("elementwise")
-    _check(lib, lib.pae_silu_mul(_ptr(out), _ptr(gate_up), tokens, (two_i // 2), block,
+    _check(lib, lib.pae_silu_mul(_ptr(out), _ptr(gate_up), tokens, (two_i // 2), block, GATE_KINDS[gate],
                                  (_code(gate_up)), _stream()))
     return out
 
@@ -831,8 +836,8 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor | N
     return both.reshape(2 * inter, k).contiguous()
 
 
-def linear_swiglu(x, weight) -> torch.Tensor:
-    """silu(x . Wg^T) * (x . Wu^T) -> [M, I] for a weight from `interleave_gate_up`. With many
+def linear_swiglu(x, weight, gate: str = "silu") -> torch.Tensor:
+    """act(x . Wg^T) (`gate`: "silu" or "relu") * (x . Wu^T) -> [M, I] for a weight from `interleave_gate_up`. With many
     tokens the activation runs in the product's epilogue; with few, in the kernel that sums the
     splits; otherwise as a kernel of its own. Gate and up are rounded to the engine dtype first in
     every one of them, so all give the same bits."""
@@ -843,7 +848,7 @@ def linear_swiglu(x, weight) -> torch.Tensor:
         out = torch.empty((source.shape[0], weight.shape[0] // 2), dtype=torch.bfloat16, device=source.device)
         lib = _lib("gemv_mma")
         _check(lib, lib.pae_linear_swiglu_few_tokens(_ptr(out), _ptr(source), _ptr(weight), _ptr(norm_weight), eps,
-                                                     source.shape[0], weight.shape[0], weight.shape[1],
+                                                     source.shape[0], weight.shape[0], weight.shape[1], GATE_KINDS[gate],
                                                      _ptr(_error_flag(source.device)), _stream()))
         return out
     x = materialized(x)
@@ -855,10 +860,10 @@ def linear_swiglu(x, weight) -> torch.Tensor:
         _need(weight, "linear_swiglu: weight")
         out = torch.empty((m, n // 2), dtype=x.dtype, device=x.device)
         lib = _lib("gemm_tcgen05")
-        _check(lib, lib.pae_linear_swiglu_tcgen05(_ptr(out), _ptr(x), _ptr(weight), m, n, k,
+        _check(lib, lib.pae_linear_swiglu_tcgen05(_ptr(out), _ptr(x), _ptr(weight), m, n, k, GATE_KINDS[gate],
                                                   _ptr(_error_flag(x.device)), _stream()))
         return out
-    return silu_mul(linear(x, weight), SWIGLU_BLOCK)
+    return silu_mul(linear(x, weight), SWIGLU_BLOCK, gate)
 
 
 def sample(logits, temperature, seed_lo, seed_hi, request_key, output_index, keep=None) -> torch.Tensor:
@@ -1003,7 +1008,7 @@ def softcap(logits, cap: float) -> torch.Tensor:
 
 def head_prep(proj, *, q_off: int, k_off: int, v_off: int, heads: int, kv_heads: int, q_dim: int, k_dim: int, value_dim: int,
               q_norm, k_norm, q_span: int, k_span: int, eps: float, table, interleaved: bool, q_rot0: int, k_rot0: int,
-              slots, keys, values, page_size: int, out_dtype, whole: bool = False) -> torch.Tensor:
+              slots, keys, values, page_size: int, out_dtype, whole: bool = False, q_out=None, direct: bool = False) -> torch.Tensor:
     """From a fused projection [tokens, ld] to attention's operands (csrc/head_prep.cu): every
     query head (q_dim channels at q_off) and key head (k_dim channels at k_off) is RMS-normed over
     its first q_span / k_span channels with the weight q_norm / k_norm (None: not normed; `whole`:
@@ -1011,12 +1016,14 @@ def head_prep(proj, *, q_off: int, k_off: int, v_off: int, heads: int, kv_heads:
     those projections), the span
     of `table.shape[1]` channels from q_rot0 / k_rot0 is rotated by the table (pairs (i, i + half),
     or (2i, 2i + 1) when `interleaved`), the queries are returned as [tokens, heads * q_dim] in
-    `out_dtype`, and keys and values (value_dim channels at v_off; `values` None: none) are written
-    to their pages at `slots` (None: nothing is written and kv_heads is ignored)."""
+    `out_dtype` (or written to the leading columns of `q_out` [tokens, >= heads * q_dim]), and keys and
+    values (value_dim channels at v_off; `values` None: none) are written to their pages at `slots`
+    (None: nothing is written and kv_heads is ignored); `direct`: they are rows [tokens, kv_heads * dim]
+    without pages."""
     proj = materialized(proj)
     _need(proj, "head_prep: projection")
     tokens, ld = proj.shape
-    writes = slots is not None and kv_heads > 0
+    writes = (slots is not None or direct) and kv_heads > 0
     need = max(q_off + heads * q_dim, (k_off + kv_heads * k_dim) if writes else 0,
                (v_off + kv_heads * value_dim) if writes and values is not None else 0)
     if need > ld:
@@ -1033,36 +1040,43 @@ def head_prep(proj, *, q_off: int, k_off: int, v_off: int, heads: int, kv_heads:
             raise KernelError(f"head_prep: a table of {table.shape[0]} rows for {tokens} tokens")
         dims = int(table.shape[1])
     if writes:
-        _need(slots, "head_prep: slots", torch.int32)
+        if not direct:
+            _need(slots, "head_prep: slots", torch.int32)
+        elif keys.numel() < tokens * kv_heads * k_dim or (values is not None and values.numel() < tokens * kv_heads * value_dim):
+            raise KernelError(f"head_prep: rows of keys or values are too few for {tokens} tokens")
         _need(keys, "head_prep: keys", out_dtype)
         if values is not None:
             _need(values, "head_prep: values", out_dtype)
-    q = torch.empty((tokens, heads * q_dim), dtype=out_dtype, device=proj.device)
+    q = q_out if q_out is not None else torch.empty((tokens, heads * q_dim), dtype=out_dtype, device=proj.device)
+    _need(q, "head_prep: queries", out_dtype)
     lib = _lib("head_prep")
-    _set_bounds("head_prep", keys if writes else None)
+    _set_bounds("head_prep", keys if writes and not direct else None)
     _check(lib, lib.pae_head_prep(
-        _ptr(q), _ptr(keys if writes else None), _ptr(values if writes else None), _ptr(proj), ld, q_off, k_off, v_off, tokens,
+        _ptr(q), q.shape[1], _ptr(keys if writes else None), _ptr(values if writes else None), _ptr(proj), ld, q_off, k_off, v_off, tokens,
         heads, kv_heads if writes else 0, q_dim, k_dim, value_dim if values is not None else 0, _ptr(q_norm), q_span,
         _ptr(k_norm), k_span, float(eps), _ptr(table), dims, 1 if interleaved else 0, q_rot0, k_rot0,
-        _ptr(slots if writes else None), page_size, 1 if whole else 0, _code(proj), _DTYPE_CODE[out_dtype], _stream()))
+        _ptr(slots if writes and not direct else None), page_size, 1 if whole else 0, 1 if direct else 0, _code(proj), _DTYPE_CODE[out_dtype], _stream()))
     return q
 
 
-def sigmoid_gate(x, gate_proj, gate_off: int, group: int = 1) -> torch.Tensor:
-    """x * sigmoid(gate_proj[:, gate_off : gate_off + x.shape[1] / group]): a gate column for every
-    `group` neighbouring channels of x (1: a gate per channel; a head's size: a gate per head)."""
+def sigmoid_gate(x, gate_proj, gate_off: int, group: int = 1, mult: float = 1.0, out=None, out_off: int = 0) -> torch.Tensor:
+    """mult * x * sigmoid(gate_proj[:, gate_off : gate_off + x.shape[1] / group]): a gate column for every
+    `group` neighbouring channels of x (1: a gate per channel; a head's size: a gate per head). With
+    `out` the result is its columns from `out_off` on."""
     x = materialized(x)
     gate_proj = materialized(gate_proj)
     _need(x, "sigmoid_gate: x")
     _need(gate_proj, "sigmoid_gate: gate")
     if gate_proj.shape[0] != x.shape[0]:
         raise KernelError(f"sigmoid_gate: {x.shape[0]} rows and {gate_proj.shape[0]} rows of gates")
-    out = torch.empty_like(x)
+    if out is None:
+        out = torch.empty_like(x)
+    _need(out, "sigmoid_gate: output", x.dtype)
     lib = _lib("head_prep")
     if group < 1 or x.shape[1] % group:
         raise KernelError(f"sigmoid_gate: rows of {x.shape[1]} channels do not split into groups of {group}")
-    _check(lib, lib.pae_sigmoid_gate(_ptr(out), _ptr(x), _ptr(gate_proj), x.shape[0], x.shape[1], gate_proj.shape[1], gate_off,
-                                     group, _code(x), _code(gate_proj), _stream()))
+    _check(lib, lib.pae_sigmoid_gate(_ptr(out), out.shape[1], out_off, _ptr(x), _ptr(gate_proj), x.shape[0], x.shape[1],
+                                     gate_proj.shape[1], gate_off, group, float(mult), _code(x), _code(gate_proj), _stream()))
     return out
 
 
@@ -1353,26 +1367,31 @@ def delta_rule(proj, offsets, w_pre, w0, a_bias, gate_offset, norm_weight, state
 # ----------------------------------------------------------------------------------- #
 # Norms without statistics around both sides of a sublayer (csrc/dyt.cu)
 
-def _dyt_step(pending, next_norm, out_dtype):
+def _dyt_step(pending, next_norm, out_dtype, next_norm2=None):
     """Runs the sum of a PendingResidual (or, for a plain tensor, nothing) and, with `next_norm` =
     (alpha, weight, bias), the Dynamic Tanh of the result in `out_dtype`: one kernel. Keeps the new
-    stream in `pending.value` and returns the normed rows or None."""
+    stream in `pending.value` and returns the normed rows or None; with `next_norm2`, a second norm
+    of the same stream, a pair of them."""
     if isinstance(pending, PendingResidual):
         x, y, post, mult, extra = materialized(pending.x), pending.y, pending.post, pending.mult, materialized(pending.extra)
+        y2 = pending.y2
     else:
-        x, y, post, mult, extra = pending, None, None, 0.0, None
+        x, y, post, mult, extra, y2 = pending, None, None, 0.0, None, None
     _need(x, "dyt: the stream", torch.float32)
     tokens, width = x.shape
-    planes = 1
+    planes = planes2 = 1
     if y is not None:
         y, planes = _sublayer_output(y)
-        if tuple(y.shape[-2:]) != (tokens, width):
-            raise KernelError(f"dyt: a sublayer's output {tuple(y.shape)} for a stream {tuple(x.shape)}")
+    if y2 is not None:
+        y2, planes2 = _sublayer_output(y2)
+    for out in (y, y2):
+        if out is not None and tuple(out.shape[-2:]) != (tokens, width):
+            raise KernelError(f"dyt: a sublayer's output {tuple(out.shape)} for a stream {tuple(x.shape)}")
     if extra is not None:
         _need(extra, "dyt: the joining stream", torch.float32)
         if tuple(extra.shape) != (tokens, width):
             raise KernelError(f"dyt: a joining stream {tuple(extra.shape)} for a stream {tuple(x.shape)}")
-    for name, norm in (("the norm after the sublayer", post), ("the next norm", next_norm)):
+    for name, norm in (("the norm after the sublayer", post), ("the next norm", next_norm), ("the second norm", next_norm2)):
         if norm is not None:
             alpha, weight, bias = norm
             _need(alpha, f"dyt: alpha of {name}", torch.float32)
@@ -1381,19 +1400,22 @@ def _dyt_step(pending, next_norm, out_dtype):
                 raise KernelError(f"dyt: {name} has {weight.numel()} weights for rows of {width}")
             if bias is not None:
                 _need(bias, f"dyt: bias of {name}", torch.float32)
-    writes = y is not None or extra is not None
+    writes = y is not None or y2 is not None or extra is not None
     x_new = torch.empty_like(x) if writes else None
     normed = torch.empty((tokens, width), dtype=out_dtype, device=x.device) if next_norm is not None else None
+    normed2 = torch.empty((tokens, width), dtype=out_dtype, device=x.device) if next_norm2 is not None else None
     post = post or (None, None, None)
     nxt = next_norm or (None, None, None)
+    nxt2 = next_norm2 or (None, None, None)
     if writes or normed is not None:
         lib = _lib("dyt")
-        _check(lib, lib.pae_dyt_step(_ptr(x_new), _ptr(normed), _ptr(x), _ptr(y), planes, _ptr(extra), _ptr(post[0]), _ptr(post[1]),
-                                     _ptr(post[2]), float(mult), _ptr(nxt[0]), _ptr(nxt[1]), _ptr(nxt[2]), tokens, width,
+        _check(lib, lib.pae_dyt_step(_ptr(x_new), _ptr(normed), _ptr(normed2), _ptr(x), _ptr(y), planes, _ptr(y2), planes2, _ptr(extra),
+                                     _ptr(post[0]), _ptr(post[1]), _ptr(post[2]), float(mult), _ptr(nxt[0]), _ptr(nxt[1]), _ptr(nxt[2]),
+                                     _ptr(nxt2[0]), _ptr(nxt2[1]), _ptr(nxt2[2]), tokens, width,
                                      _DTYPE_CODE[out_dtype] if out_dtype is not None else 0, _stream()))
     if isinstance(pending, PendingResidual):
         pending.value = x_new if writes else x
-    return normed
+    return normed if next_norm2 is None else (normed, normed2)
 
 
 def dyt_norm(x, alpha, weight, bias, out_dtype) -> torch.Tensor:
@@ -1407,10 +1429,21 @@ def dyt_norm(x, alpha, weight, bias, out_dtype) -> torch.Tensor:
     return _dyt_step(x, (alpha, weight, bias), out_dtype)
 
 
-def residual_add(x, y, mult: float = 1.0, post=None):
-    """The stream x + mult * post(y), float32, pending: `post` = (alpha, weight, bias) of a Dynamic Tanh
-    over y, or None. The next `dyt_norm` makes the sum in its own kernel."""
-    return PendingResidual(x, y, post, mult)
+def dyt_norm_pair(x, first, second, out_dtype):
+    """Two Dynamic Tanh norms, each (alpha, weight, bias), of the same stream in one pass over it: what
+    two sublayers side by side read. x as for `dyt_norm`; a pending sum is made on the way."""
+    if not (isinstance(x, PendingResidual) and x.value is None):
+        x = materialized(x)
+        if x.dtype != torch.float32:
+            raise KernelError(f"dyt_norm_pair: the stream is {x.dtype}, float32 is needed")
+    return _dyt_step(x, first, out_dtype, second)
+
+
+def residual_add(x, y, mult: float = 1.0, post=None, y2=None):
+    """The stream x + mult * post(y) (+ y2), float32, pending: `post` = (alpha, weight, bias) of a Dynamic
+    Tanh over y, or None; `y2` the output of a second sublayer that ran beside the first. The next
+    `dyt_norm` makes the sum in its own kernel."""
+    return PendingResidual(x, y, post, mult, y2=y2)
 
 
 def join_stream(x, extra):
@@ -1420,6 +1453,144 @@ def join_stream(x, extra):
         x.extra = extra
         return x
     return PendingResidual(materialized(x), None, None, 0.0, extra)
+
+
+# ----------------------------------------------------------------------------------- #
+# A memory that decays (csrc/decay_memory.cu) and what stands around it (csrc/state_space.cu)
+
+def _state_rows(state, floats: int, what: str):
+    """(address, floats between slots) of per-request state of `floats` float32 numbers a slot; the slots
+    may be rows of something wider."""
+    if not state.is_cuda or state.dtype != torch.float32:
+        raise KernelError(f"{what}: the state is {state.dtype} on {state.device}")
+    if state.dim() < 2 or not state[0].is_contiguous() or state[0].numel() != floats:
+        raise KernelError(f"{what}: state rows are {tuple(state.shape[1:])}, {floats} numbers are needed")
+    return state.data_ptr(), int(state.stride(0))
+
+
+def decay_memory(q, k, v, state, q_start, state_slot, num_seqs: int, num_heads: int, groups: int, key_dim: int, value_dim: int,
+                 log_decay=None, head_decay=None, step=None, k_scale: float = 1.0, skip=None, max_q_len: int = 1,
+                 num_single: int | None = None, multi_index=None, form: str | None = None) -> torch.Tensor:
+    """S <- a S + (w k) v^T, o = S^T q (+ skip v) over the step's tokens, from and into the per-request
+    state (float32, [heads, key_dim, value_dim] a slot): see csrc/decay_memory.cu. q, k and v are
+    (tensor [tokens, ld], first column): `groups` query and key heads, `num_heads` value heads. a =
+    exp(log_decay [tokens, heads]) or head_decay [heads]; w = step [tokens, heads] or k_scale. Single
+    tokens take the step kernel, portions the chunked tensor-core kernels (bfloat16, rows of
+    16-byte pieces), everything else, and everything when `form` is "scan", goes token after token.
+    -> float32 [tokens, heads * value_dim]."""
+    tokens = q[0].shape[0]
+    rows = []
+    for name, (t, off), width in (("q", q, groups * key_dim), ("k", k, groups * key_dim), ("v", v, num_heads * value_dim)):
+        _need(t, f"decay_memory: {name}", q[0].dtype)
+        if t.dim() != 2 or t.shape[0] != tokens or off < 0 or off + width > t.shape[1]:
+            raise KernelError(f"decay_memory: {name} columns {off}..{off + width} of {tuple(t.shape)} for {tokens} tokens")
+        rows += [t.data_ptr() + off * t.element_size(), int(t.shape[1])]
+    if (log_decay is None) == (head_decay is None):
+        raise KernelError("decay_memory: one of log_decay and head_decay is needed")
+    for name, t, n in (("log_decay", log_decay, tokens * num_heads), ("step", step, tokens * num_heads),
+                       ("head_decay", head_decay, num_heads), ("skip", skip, num_heads)):
+        if t is not None:
+            _need(t, f"decay_memory: {name}", torch.float32)
+            if t.numel() != n:
+                raise KernelError(f"decay_memory: {name} has {t.numel()} numbers, {n} are needed")
+    _need(q_start, "decay_memory: q_start", torch.int32)
+    _need(state_slot, "decay_memory: state_slot", torch.int32)
+    address, stride = _state_rows(state, num_heads * key_dim * value_dim, "decay_memory")
+    o = torch.empty((tokens, num_heads * value_dim), dtype=torch.float32, device=q[0].device)
+    lib = _lib("decay_memory")
+    what = (_ptr(o), address, stride, *rows, _ptr(log_decay), _ptr(head_decay), _ptr(step), float(k_scale), _ptr(skip), _ptr(q_start),
+            _ptr(state_slot))
+    sizes = (num_heads, groups, key_dim, value_dim)
+    code = _code(q[0])
+    singles = num_single if num_single is not None else (num_seqs if max_q_len == 1 else -1)
+    stepped = form != "scan" and address % 16 == 0 and lib.pae_decay_memory_step_supports(key_dim, value_dim, stride) == 1
+    if stepped and singles != 0:
+        _check(lib, lib.pae_decay_memory_step(*what, num_seqs, *sizes, code, _stream()))
+    if singles == num_seqs and stepped:
+        return o
+    chunked = (form != "scan" and use_tensor_cores and code == 1 and address % 16 == 0 and all(r % 16 == 0 for r in rows[::2])
+               and lib.pae_decay_memory_chunked_supports(key_dim, value_dim, rows[1], rows[3], rows[5], stride) == 1)
+    if not chunked or not stepped:
+        _check(lib, lib.pae_decay_memory_scan(*what, num_seqs, *sizes, 1 if stepped else 0, code, _stream()))
+        return o
+    listed = num_seqs
+    if multi_index is not None:
+        _need(multi_index, "decay_memory: multi_index", torch.int32)
+        listed = multi_index.numel()
+    slots = tokens // lib.pae_decay_memory_chunk() + listed
+    size = num_heads * key_dim * value_dim
+    contribution = torch.empty(slots * size, dtype=torch.float32, device=o.device)
+    before = torch.empty(slots * 2 * size, dtype=torch.bfloat16, device=o.device)
+    decay = torch.empty(slots * num_heads, dtype=torch.float32, device=o.device)
+    _check(lib, lib.pae_decay_memory_chunked(*what, _ptr(multi_index), listed, max_q_len, *sizes, _ptr(contribution), _ptr(before),
+                                             _ptr(decay), _stream()), 3)
+    return o
+
+
+def ssm_prepare(proj, z_off: int, z_cols: int, u_off: int, channels: int, dt_off: int, heads: int, taps_weight, bias, dt_bias, a_log,
+                state, q_start, q_pos0, state_slot, num_seqs: int, max_q_len: int, out_dtype):
+    """From the fused input projection (float32 [tokens, ld], or the planes of a split product) of a
+    selective state space to its recurrence's operands (csrc/state_space.cu): -> (u = silu(causal
+    convolution of the `channels` columns at u_off) [tokens, channels] in `out_dtype`, step =
+    softplus(dt + dt_bias) and log_decay = -exp(a_log) step, float32 [tokens, heads], and the gate as
+    (rows, first column): the projection itself, or its summed columns). `state` float32 [slots, (taps - 1) *
+    channels] is brought up to date."""
+    proj, planes = _sublayer_output(proj)
+    tokens, ld = int(proj.shape[-2]), int(proj.shape[-1])
+    for off, width in ((z_off, z_cols), (u_off, channels), (dt_off, heads)):
+        if off < 0 or off + width > ld:
+            raise KernelError(f"ssm_prepare: columns {off}..{off + width} of rows of {ld}")
+    _need(taps_weight, "ssm_prepare: taps", torch.float32)
+    if taps_weight.dim() != 2 or taps_weight.shape[0] != channels:
+        raise KernelError(f"ssm_prepare: taps are {tuple(taps_weight.shape)} for {channels} channels")
+    taps = int(taps_weight.shape[1])
+    for name, t, n in (("bias", bias, channels), ("dt_bias", dt_bias, heads), ("a_log", a_log, heads)):
+        if t is not None:
+            _need(t, f"ssm_prepare: {name}", torch.float32)
+            if t.numel() != n:
+                raise KernelError(f"ssm_prepare: {name} has {t.numel()} numbers, {n} are needed")
+    for name, t in (("q_start", q_start), ("q_pos0", q_pos0), ("state_slot", state_slot)):
+        _need(t, f"ssm_prepare: {name}", torch.int32)
+    address, stride = None, 0
+    if taps > 1:
+        address, stride = _state_rows(state, (taps - 1) * channels, "ssm_prepare")
+    u = torch.empty((tokens, channels), dtype=out_dtype, device=proj.device)
+    step = torch.empty((tokens, heads), dtype=torch.float32, device=proj.device)
+    log_decay = torch.empty((tokens, heads), dtype=torch.float32, device=proj.device)
+    z = torch.empty((tokens, z_cols), dtype=torch.float32, device=proj.device) if planes > 1 else None
+    lib = _lib("state_space")
+    _check(lib, lib.pae_ssm_prepare(_ptr(u), _ptr(step), _ptr(log_decay), _ptr(z), address, stride, _ptr(proj), planes, ld, z_off, z_cols,
+                                    u_off, channels, dt_off, heads, _ptr(taps_weight), taps, _ptr(bias), _ptr(dt_bias), _ptr(a_log),
+                                    _ptr(q_start), _ptr(q_pos0), _ptr(state_slot), tokens, num_seqs, max_q_len,
+                                    _DTYPE_CODE[out_dtype], _stream()))
+    return u, step, log_decay, (z, 0) if z is not None else (proj.view(tokens, ld), z_off)
+
+
+def gated_group_norm(y, gate, gate_off: int, groups: int, eps: float, out_dtype, weight=None, gate_first: bool = False, mult: float = 1.0,
+                     out=None, out_off: int = 0) -> torch.Tensor:
+    """The channels of float32 rows y in `groups` equal parts, each divided by its own root mean square,
+    times silu(gate[:, gate_off ...]) before (`gate_first`) or after the division, times `weight` (or
+    none) and `mult`, in `out_dtype`; with `out`, its columns from `out_off` on."""
+    gate = materialized(gate)
+    _need(y, "gated_group_norm: y", torch.float32)
+    _need(gate, "gated_group_norm: gate", torch.float32)
+    tokens, width = y.shape
+    if groups < 1 or width % groups:
+        raise KernelError(f"gated_group_norm: rows of {width} in {groups} groups")
+    if gate.shape[0] != tokens:
+        raise KernelError(f"gated_group_norm: {tokens} rows and {gate.shape[0]} rows of gates")
+    if weight is not None:
+        _need(weight, "gated_group_norm: weight", torch.float32)
+        if weight.numel() != width:
+            raise KernelError(f"gated_group_norm: weight of {weight.numel()} for rows of {width}")
+    if out is None:
+        out = torch.empty((tokens, width), dtype=out_dtype, device=y.device)
+    _need(out, "gated_group_norm: output", out_dtype)
+    lib = _lib("state_space")
+    _check(lib, lib.pae_gated_group_norm(_ptr(out), out.shape[1], out_off, _ptr(y), _ptr(gate), gate.shape[1], gate_off, _ptr(weight), tokens,
+                                         groups, width // groups, 1 if gate_first else 0, float(eps), float(mult),
+                                         _DTYPE_CODE[out_dtype], _stream()))
+    return out
 
 
 # ----------------------------------------------------------------------------------- #

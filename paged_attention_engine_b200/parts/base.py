@@ -53,6 +53,7 @@ from ..config.model_spec import PartSpec
 class TensorSpec:
     """One checkpoint tensor. `kind` decides its storage and its random initialisation:
 
+    log_rate the logarithm of a positive rate per head: held in float32; drawn uniformly from (-2, 1).
     matrix   a weight of a matrix product: engine dtype (bfloat16 or float32);
              drawn N(0, 0.02).
     vector   a bias: held in float32; drawn N(0, 0.02).
@@ -159,6 +160,35 @@ class Part:
     @classmethod
     def state_need(cls, spec: PartSpec) -> StateNeed | None:
         return None
+
+
+class ProjectedMixer(Part):
+    """A mixer of the form W_o mix(W_in h + b_in): one product in front, one behind, and between them what
+    makes the mixer. Such mixers can also stand side by side behind one shared product on either side (see
+    `side_by_side.py`), so what is between is a method of its own.
+
+    A subclass sets `in_weight` [columns, hidden], `in_bias` (float32 [columns] or None) and `o_weight`
+    [hidden, out_width], and provides `mix(ctx, proj, offset, cache, out, out_offset, mult)`: from the
+    projection's columns [offset, offset + columns) (float32 rows, perhaps the planes of a split
+    product) to mult times the output product's operand, in the engine's dtype, written to columns
+    [out_offset, out_offset + out_width) of `out`."""
+
+    in_bias = None
+
+    @property
+    def out_width(self) -> int:
+        return int(self.o_weight.shape[1])
+
+    def mix(self, ctx, proj, offset: int, cache, out, out_offset: int, mult: float) -> None:
+        raise NotImplementedError
+
+    def forward(self, ctx, x, residual, cache):
+        ops = self.ops
+        proj = ops.linear(x, self.in_weight, self.in_bias, None, out_dtype=torch.float32)
+        out = torch.empty((proj.shape[0], self.out_width), dtype=self.runtime.dtype, device=self.runtime.device)
+        self.mix(ctx, proj, 0, cache, out, 0, 1.0)
+        # without a residual (a caller that sums by itself) the output leaves in float32
+        return ops.linear(out, self.o_weight, None, residual, out_dtype=residual.dtype if residual is not None else torch.float32)
 
 
 class Registry:

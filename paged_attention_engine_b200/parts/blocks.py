@@ -35,6 +35,35 @@ class ParallelResidual(Block):
         return layer.feed_forward.forward(ctx, normed, ctx.ops.materialized(hidden))
 
 
+@BLOCKS.register("parallel_two_norms")
+class ParallelTwoNorms(Block):
+    """Both branches read the same stream, each through a norm of its own: x <- x + mixer(norm_a(x)) +
+    ff(norm_b(x)). The branches get no residual and leave float32; the sum of the three stays pending
+    until the next norm reads the stream, and norms that can (`forward_pair`) read it together."""
+
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward"}
+
+    def forward(self, ctx, hidden, layer, cache):
+        first, second = layer.mixer_norm, layer.feed_forward_norm
+        if hasattr(first, "forward_pair") and type(first) is type(second):
+            a, b = first.forward_pair(ctx, hidden, second)
+        else:
+            a, b = first.forward(ctx, hidden), second.forward(ctx, hidden)
+        mixed = layer.mixer.forward(ctx, a, None, cache)
+        return ctx.ops.residual_add(ctx.ops.materialized(hidden), mixed, 1.0, y2=layer.feed_forward.forward(ctx, b, None))
+
+
+@BLOCKS.register("summed_mixer")
+class SummedMixer(Block):
+    """A layer without a feed-forward whose sum stays pending until the next norm: x <- x + mixer(norm(x))."""
+
+    roles = {"norm": "norm", "mixer": "mixer"}
+
+    def forward(self, ctx, hidden, layer, cache):
+        normed = layer.norm.forward(ctx, hidden)
+        return ctx.ops.residual_add(ctx.ops.materialized(hidden), layer.mixer.forward(ctx, normed, None, cache))
+
+
 @BLOCKS.register("mixer_residual")
 class MixerResidual(Block):
     """A layer without a feed-forward: x <- x + mixer(norm(x))."""

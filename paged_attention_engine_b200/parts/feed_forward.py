@@ -10,41 +10,51 @@ from ..config.model_spec import PartSpec
 from .base import FEED_FORWARDS, Part, TensorSpec
 
 
-@FEED_FORWARDS.register("swiglu")
-class SwiGLU(Part):
-    """params: hidden_size, intermediate_size. tensors: gate_proj/up_proj/down_proj .weight."""
+@FEED_FORWARDS.register("gated_mlp")
+class GatedMLP(Part):
+    """down(act(gate(x)) * up(x)) without biases. params: hidden_size, intermediate_size, activation
+    ("silu", the default, or "relu"). tensors: gate, up [intermediate, hidden], down [hidden,
+    intermediate]. The residual may be float32 while x is in the engine's dtype; without a residual (a
+    caller that sums by itself) the output leaves in float32."""
+
+    tensor_names = ("gate", "up", "down")
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec) -> list[TensorSpec]:
         hidden, inter = int(spec.params["hidden_size"]), int(spec.params["intermediate_size"])
-        return [
-            TensorSpec(spec.tensor_name("gate_proj.weight"), (inter, hidden), "matrix"),
-            TensorSpec(spec.tensor_name("up_proj.weight"), (inter, hidden), "matrix"),
-            TensorSpec(spec.tensor_name("down_proj.weight"), (hidden, inter), "matrix"),
-        ]
+        gate, up, down = (spec.tensor_name(n) for n in cls.tensor_names)
+        return [TensorSpec(gate, (inter, hidden), "matrix"), TensorSpec(up, (inter, hidden), "matrix"),
+                TensorSpec(down, (hidden, inter), "matrix")]
 
     def __init__(self, spec, tensors, runtime):
         super().__init__(spec, tensors, runtime)
         self.intermediate_size = int(spec.params["intermediate_size"])
-        gate = tensors.pop(spec.tensor_name("gate_proj.weight"))
-        up = tensors.pop(spec.tensor_name("up_proj.weight"))
+        self.activation = str(spec.params.get("activation", "silu"))
+        gate, up = (tensors.pop(spec.tensor_name(n)) for n in self.tensor_names[:2])
         # Gate and up are one product. Where the kernels offer it, their rows alternate in
-        # blocks (16 gate rows, their 16 up rows, ...) so that SiLU x up runs inside the
+        # blocks (16 gate rows, their 16 up rows, ...) so that act(gate) x up runs inside the
         # product; else rows [0, I) are the gate and rows [I, 2I) the up projection.
         interleave = getattr(self.ops, "interleave_gate_up", None)
         self.gate_up_weight = interleave(gate, up) if interleave is not None else None
         self.interleaved = self.gate_up_weight is not None
         if not self.interleaved:
             self.gate_up_weight = torch.cat([gate, up], dim=0).contiguous()
-        self.down_weight = tensors.pop(spec.tensor_name("down_proj.weight"))
+        self.down_weight = tensors.pop(spec.tensor_name(self.tensor_names[2]))
 
     def forward(self, ctx, x, residual):
         ops = self.ops
         if self.interleaved:
-            hidden = ops.linear_swiglu(x, self.gate_up_weight)
+            hidden = ops.linear_swiglu(x, self.gate_up_weight, gate=self.activation)
         else:
-            hidden = ops.silu_mul(ops.linear(x, self.gate_up_weight, None))
-        return ops.linear(hidden, self.down_weight, None, residual)
+            hidden = ops.silu_mul(ops.linear(x, self.gate_up_weight, None), gate=self.activation)
+        return ops.linear(hidden, self.down_weight, None, residual, out_dtype=residual.dtype if residual is not None else torch.float32)
+
+
+@FEED_FORWARDS.register("swiglu")
+class SwiGLU(GatedMLP):
+    """`gated_mlp` with SiLU. tensors: gate_proj/up_proj/down_proj .weight."""
+
+    tensor_names = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
 
 
 @FEED_FORWARDS.register("dense_mlp")

@@ -1,9 +1,9 @@
 """Grouped-query attention with normed, partly rotated heads, a sink and an output gate.
 
-q, k, v and the gate are one fused projection without bias (float32 out). Every query and key
-head is RMS-normed over its channels with a weight that all heads share (or all query heads of a
+q, k, v and the gate are one fused projection (float32 out), q, k and v with or without biases. Every
+query and key head may be RMS-normed over its channels with a weight that all heads share (or all query heads of a
 token are normed at once, and all its key heads, with weights as long as those projections), then
-a leading span of the head is rotated (pairs (i, i + span/2)) by the layer's position encoding;
+a leading span of the head is rotated (pairs (i, i + span/2), or neighbours (2i, 2i + 1)) by the layer's position encoding;
 keys and values go to their pages. Query i sees key j <= i with i - j < window (no window: every
 earlier key). The softmax's denominator may hold one more term exp(s_h) without a value (a sink:
 s_h = 0, or a learned number per head), and the concatenated heads may be multiplied by
@@ -16,18 +16,19 @@ from __future__ import annotations
 import torch
 
 from ..config.model_spec import PartSpec
-from .base import MIXERS, CacheNeed, Part, TensorSpec
+from .base import MIXERS, CacheNeed, ProjectedMixer, TensorSpec
 
 
 @MIXERS.register("gated_window_attention")
-class GatedWindowAttention(Part):
+class GatedWindowAttention(ProjectedMixer):
     """params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim, scale, window (0: all
     keys), qk_norm_eps (None: q and k are not normed), qk_norm ("head", the default: per head with a
     weight [head_dim] that the heads share; "whole": over the whole projection with weights [heads *
     head_dim] and [kv_heads * head_dim]), unit_sink (bool), learned_sink (bool: a tensor `sink`
     [heads]), output_gate (False, True or "channel": g [heads * value_dim, hidden]; "head": g [heads,
-    hidden]), position_encoding (a dict with its `kind` and `dims`, or None).
-    tensors: q, k, v, o (and g) matrices; q.norm, k.norm; sink."""
+    hidden]), qkv_bias (bool: q.b, k.b, v.b, added in the projection), pairing ("half", the default, or
+    "interleaved": which channels rotate together), position_encoding (a dict with its `kind` and `dims`,
+    or None). tensors: q, k, v, o (and g) matrices; q.b, k.b, v.b; q.norm, k.norm; sink."""
 
     @classmethod
     def _sizes(cls, spec: PartSpec):
@@ -44,6 +45,8 @@ class GatedWindowAttention(Part):
         if p.get("output_gate"):
             rows["g"] = heads if p["output_gate"] == "head" else heads * dv
         out = [TensorSpec(spec.tensor_name(n), (r, hidden), "matrix") for n, r in rows.items()]
+        if p.get("qkv_bias"):
+            out += [TensorSpec(spec.tensor_name(f"{n}.b"), (rows[n],), "vector") for n in ("q", "k", "v")]
         if p.get("qk_norm_eps") is not None:
             whole = p.get("qk_norm", "head") == "whole"
             out += [TensorSpec(spec.tensor_name("q.norm"), (heads * d if whole else d,), "scale"),
@@ -82,6 +85,13 @@ class GatedWindowAttention(Part):
         names = ("q", "k", "v") + (("g",) if self.gated else ())
         # One projection for q | k | v | g: the columns of its output in that order.
         self.in_weight = torch.cat([tensors.pop(spec.tensor_name(n)) for n in names], dim=0).contiguous()
+        if p.get("qkv_bias"):
+            biases = [tensors.pop(spec.tensor_name(f"{n}.b")) for n in ("q", "k", "v")]
+            gate_columns = self.in_weight.shape[0] - sum(b.numel() for b in biases)          # the gate has none
+            self.in_bias = torch.cat(biases + [biases[0].new_zeros(gate_columns)]).contiguous()
+        if p.get("pairing", "half") not in ("half", "interleaved"):
+            raise ValueError(f"gated_window_attention: pairing '{p.get('pairing')}' (half, interleaved)")
+        self.interleaved = p.get("pairing", "half") == "interleaved"
         self.q_norm = self.k_norm = None
         if self.norm_eps is not None:
             self.q_norm, self.k_norm = tensors.pop(spec.tensor_name("q.norm")), tensors.pop(spec.tensor_name("k.norm"))
@@ -96,22 +106,33 @@ class GatedWindowAttention(Part):
         if self.rot_dims > self.head_dim:
             raise ValueError(f"gated_window_attention: {self.rot_dims} rotated channels in heads of {self.head_dim}")
 
-    def forward(self, ctx, x, residual, cache):
+    def _attend(self, ctx, proj, offset, cache):
+        """[tokens, heads * value_dim]: every head's softmax average, before the gate."""
         ops = self.ops
         group = ctx.groups[cache.group]
         h, g, d, dv = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim
-        proj = ops.linear(x, self.in_weight, None, None, out_dtype=torch.float32)
         table = self.position_encoding.table(ctx) if self.position_encoding is not None else None
         q = ops.head_prep(
-            proj, q_off=0, k_off=h * d, v_off=(h + g) * d, heads=h, kv_heads=g, q_dim=d, k_dim=d, value_dim=dv,
+            proj, q_off=offset, k_off=offset + h * d, v_off=offset + (h + g) * d, heads=h, kv_heads=g, q_dim=d, k_dim=d, value_dim=dv,
             q_norm=self.q_norm, k_norm=self.k_norm, q_span=d, k_span=d, eps=float(self.norm_eps or 0.0),
-            table=table, interleaved=False, q_rot0=0, k_rot0=0, slots=group.slots if cache.writes else None,
+            table=table, interleaved=self.interleaved, q_rot0=0, k_rot0=0, slots=group.slots if cache.writes else None,
             keys=cache.keys, values=cache.values, page_size=cache.page_size, out_dtype=self.runtime.dtype, whole=self.whole_norm)
-        out = ops.paged_attention_scored(
+        return ops.paged_attention_scored(
             q, cache.keys, cache.values, group.block_table, ctx.q_start, ctx.q_pos0, ctx.kv_len, h, g, d, dv,
             cache.page_size, ctx.max_q_len, self.scale, sink=self.sink, window=self.window,
             max_kv_len=ctx.max_kv_len, num_single=ctx.num_single)
+
+    def mix(self, ctx, proj, offset, cache, out, out_offset, mult):
+        if not self.gated:
+            raise ValueError("gated_window_attention: without a gate the heads cannot stand beside another mixer")
+        proj = self.ops.materialized(proj)
+        gate_off = offset + (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.value_dim
+        self.ops.sigmoid_gate(self._attend(ctx, proj, offset, cache), proj, gate_off, group=self.gate_group, mult=mult, out=out, out_off=out_offset)
+
+    def forward(self, ctx, x, residual, cache):
         if self.gated:
-            out = ops.sigmoid_gate(out, proj, (h + g) * d + g * dv, group=self.gate_group)
-        # without a residual (a caller that sums by itself) the output leaves in float32
-        return ops.linear(out, self.o_weight, None, residual, out_dtype=residual.dtype if residual is not None else torch.float32)
+            return super().forward(ctx, x, residual, cache)
+        ops = self.ops
+        proj = ops.materialized(ops.linear(x, self.in_weight, self.in_bias, None, out_dtype=torch.float32))
+        return ops.linear(self._attend(ctx, proj, 0, cache), self.o_weight, None, residual,
+                          out_dtype=residual.dtype if residual is not None else torch.float32)

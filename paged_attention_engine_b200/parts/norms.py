@@ -112,6 +112,10 @@ class DynamicTanh(Part):
     def forward(self, ctx, x):
         return self.ops.dyt_norm(x, self.alpha, self.weight, self.bias, self.runtime.dtype)
 
+    def forward_pair(self, ctx, x, other: "DynamicTanh"):
+        """This norm and another one of the same stream, in one pass over it."""
+        return self.ops.dyt_norm_pair(x, (self.alpha, self.weight, self.bias), (other.alpha, other.weight, other.bias), self.runtime.dtype)
+
     def add_to(self, ctx, stream, y, mult: float):
         """stream + mult * norm(y): float32, pending until the next read."""
         return self.ops.residual_add(stream, y, mult, (self.alpha, self.weight, self.bias))

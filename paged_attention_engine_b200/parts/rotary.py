@@ -75,8 +75,8 @@ def ramped_frequencies(freqs, dims: int, base: float, factor: float, original: f
 class ScaledRotary(Part):
     """Cosines and sines for a rotated span of `dims` channels, with the frequencies base^(-2i/dims)
     rescaled for sequences longer than the ones the frequencies were made for. params: dims, base,
-    scaling: None, or {"kind": "banded", factor, low, high, original}, or {"kind": "ramped",
-    factor, original, fast, slow}. No tensors. The frequencies are worked out in double
+    scaling: None, or {"kind": "linear", factor} (every frequency divided by it), or {"kind": "banded",
+    factor, low, high, original}, or {"kind": "ramped", factor, original, fast, slow}. No tensors. The frequencies are worked out in double
     precision and rounded once to float32; the angle is a float32 product on the device. Which
     channels the span covers and how they pair is the mixer's business."""
 
@@ -92,12 +92,14 @@ class ScaledRotary(Part):
         scaling = p.get("scaling")
         if scaling is not None:
             s = {k: float(v) for k, v in scaling.items() if k != "kind"}
-            if scaling.get("kind") == "banded":
+            if scaling.get("kind") == "linear":
+                freqs = [f / s["factor"] for f in freqs]
+            elif scaling.get("kind") == "banded":
                 freqs = banded_frequencies(freqs, s["factor"], s["low"], s["high"], s["original"])
             elif scaling.get("kind") == "ramped":
                 freqs, self.amplitude = ramped_frequencies(freqs, self.dims, self.base, s["factor"], s["original"], s["fast"], s["slow"])
             else:
-                raise ValueError(f"scaled_rotary: scaling kind {scaling.get('kind')!r} (banded, ramped)")
+                raise ValueError(f"scaled_rotary: scaling kind {scaling.get('kind')!r} (linear, banded, ramped)")
         self.inv_freq = torch.tensor(freqs, dtype=torch.float64).to(torch.float32).to(runtime.device)
         self._key = ("scaled_rotary", self.dims, self.base, tuple(sorted((scaling or {}).items())))
 

@@ -70,11 +70,12 @@ def _checkpoint_files(folder: Path) -> list[Path]:
 
 
 def check_against_specs(
-    expected: dict[str, TensorSpec], present: dict[str, tuple[int, ...]], where: str
+    expected: dict[str, TensorSpec], present: dict[str, tuple[int, ...]], where: str, unread: Iterable[str] = ()
 ) -> None:
-    """Raises one error that lists missing and unexpected tensors and wrong shapes."""
+    """Raises one error that lists missing and unexpected tensors and wrong shapes; `unread` names may be
+    present without being read."""
     missing = [n for n in expected if n not in present]
-    unexpected = [n for n in present if n not in expected]
+    unexpected = [n for n in present if n not in expected and n not in set(unread)]
     wrong = [
         f"{n}: file has {tuple(present[n])}, the model reads {tuple(expected[n].shape)}"
         for n in expected
@@ -100,7 +101,7 @@ def place(tensor: torch.Tensor, spec: TensorSpec, dtype: torch.dtype, device) ->
         return tensor.to(device=device, dtype=torch.int32).contiguous()
     if not tensor.dtype.is_floating_point:
         raise WeightsError(f"{spec.name}: stored as {tensor.dtype}, a floating-point tensor is read")
-    if spec.kind in ("vector", "scale", "taps", "rate", "mixing"):
+    if spec.kind in ("vector", "scale", "taps", "rate", "mixing", "log_rate"):
         return tensor.to(device=device, dtype=torch.float32).contiguous()
     if dtype == torch.bfloat16 and tensor.dtype in (torch.float32, torch.float64):
         return tensor.to(device=device, dtype=torch.float32).contiguous()
@@ -123,12 +124,12 @@ def load_tensors(folder: str | Path, spec: ModelSpec, dtype: torch.dtype, device
             for name in f.keys():
                 present[name] = tuple(f.get_slice(name).get_shape())
                 owner[name] = path
-    check_against_specs(expected, present, str(folder))
+    check_against_specs(expected, present, str(folder), spec.unread)
     out: dict[str, torch.Tensor] = {}
     for path in files:
         with safe_open(str(path), framework="pt", device="cpu") as f:
             for name in f.keys():
-                if owner[name] == path:
+                if owner[name] == path and name in expected:
                     out[name] = place(f.get_tensor(name), expected[name], dtype, device)
     return out
 
@@ -138,8 +139,8 @@ def place_tensors(
 ) -> dict[str, torch.Tensor]:
     """The same validation and placement for tensors that are already in memory."""
     expected = collect_tensor_specs(spec)
-    check_against_specs(expected, {n: tuple(t.shape) for n, t in tensors.items()}, where)
-    return {n: place(t, expected[n], dtype, device) for n, t in tensors.items()}
+    check_against_specs(expected, {n: tuple(t.shape) for n, t in tensors.items()}, where, spec.unread)
+    return {n: place(t, expected[n], dtype, device) for n, t in tensors.items() if n in expected}
 
 
 def names_in(files: Iterable[Path]) -> list[str]:

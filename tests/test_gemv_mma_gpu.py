@@ -59,7 +59,7 @@ def _linear(ops, x, w, residual=None, norm=None, eps=0.0):
 
 def _swiglu(ops, x, w, norm=None, eps=0.0):
     out = torch.empty((x.shape[0], w.shape[0] // 2), dtype=torch.bfloat16, device="cuda")
-    _call(ops, "pae_linear_swiglu_few_tokens", _ptr(out), _ptr(x), _ptr(w), _ptr(norm), eps, x.shape[0], w.shape[0], w.shape[1],
+    _call(ops, "pae_linear_swiglu_few_tokens", _ptr(out), _ptr(x), _ptr(w), _ptr(norm), eps, x.shape[0], w.shape[0], w.shape[1], 0,
           _flag(ops), 0)
     return out
 

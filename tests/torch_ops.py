@@ -100,10 +100,10 @@ def paged_attention(
     return out.view(tokens, num_heads * head_dim).to(qkv.dtype)
 
 
-def silu_mul(gate_up):
+def silu_mul(gate_up, block=0, gate="silu"):
     half = gate_up.shape[-1] // 2
-    gate, up = gate_up[..., :half].float(), gate_up[..., half:].float()
-    return (torch.nn.functional.silu(gate) * up).to(gate_up.dtype)
+    g, up = gate_up[..., :half].float(), gate_up[..., half:].float()
+    return ((torch.nn.functional.silu(g) if gate == "silu" else g.clamp_min(0.0)) * up).to(gate_up.dtype)
 
 
 def gather_rows(x, rows):
