@@ -8,6 +8,10 @@
 // retention of a fixed decay per head and Mamba-2's selective state space are both this
 // recurrence. The state is float32 [n][dv] per request and head, carried from token to token.
 //
+// For float32 operands the arithmetic of `scan` and `step` is double: a read-out sums n products of a
+// state that itself sums a thousand tokens, and where the sum cancels, the norm that follows
+// multiplies what float32 sums would have lost. The state between two calls is float32 always.
+//
 // Three ways through it, which give the same numbers up to rounding:
 //
 //   scan     token after token, any sizes up to 1,024 key channels, float32 or bfloat16 operands. A
@@ -60,16 +64,30 @@ struct Memory {
 // ---------------------------------------------------------------------------------------
 constexpr int SCAN_WARPS = 4;
 
+// The type in which a recurrence over operands of type T is carried within a call.
+template <typename T>
+struct Carried {
+  using type = double;
+};
+template <>
+struct Carried<__nv_bfloat16> {
+  using type = float;
+};
+__device__ __forceinline__ float exp_of(float x) { return expf(x); }
+__device__ __forceinline__ double exp_of(double x) { return exp(x); }
+
 template <typename T, int PER, int KS>
 __global__ void __launch_bounds__(SCAN_WARPS * 32) memory_scan_kernel(const Memory p) {
   dependent_launch_prologue();
+  using A = typename Carried<T>::type;
   constexpr int TILE = KS >= 16 ? 4 : 16;    // tokens at a time in shared memory
   constexpr int SEG = PER + 4;               // a part's channels in shared memory, padded against bank conflicts
   constexpr int ROW = KS * SEG;
   constexpr int WARP_COLS = 32 / KS, COLS = SCAN_WARPS * WARP_COLS;
   __shared__ __align__(16) float qs[TILE][ROW];
   __shared__ __align__(16) float ks[TILE][ROW];
-  __shared__ float vs[TILE][COLS], keep[TILE], add[TILE];
+  __shared__ float vs[TILE][COLS], add[TILE];
+  __shared__ A keep[TILE];
   const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * COLS;
   const int first = p.q_start[b], count = p.q_start[b + 1] - first;
   if (count <= 0 || (p.skip_single && count == 1)) return;
@@ -78,14 +96,14 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) memory_scan_kernel(const Memo
   const int part = lane / WARP_COLS, local = warp * WARP_COLS + lane % WARP_COLS, col = c0 + local;
   const bool has_col = col < dv;
   float* st = p.state + (size_t)p.state_slot[b] * p.slot_stride + (size_t)h * n * dv;
-  float s[PER];
+  A s[PER];
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int row = part * PER + i;
-    s[i] = has_col && row < n ? st[(size_t)row * dv + col] : 0.f;
+    s[i] = has_col && row < n ? (A)st[(size_t)row * dv + col] : (A)0;
   }
-  const float skip = p.skip != nullptr ? p.skip[h] : 0.f;
-  const float fixed = p.log_decay == nullptr ? p.head_decay[h] : 0.f;
+  const A skip = p.skip != nullptr ? p.skip[h] : 0.f;
+  const A fixed = p.log_decay == nullptr ? p.head_decay[h] : 0.f;
   for (int t0 = 0; t0 < count; t0 += TILE) {
     const int tokens = min(TILE, count - t0);
     __syncthreads();
@@ -101,38 +119,38 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) memory_scan_kernel(const Memo
     }
     if (tid < tokens) {
       const size_t at = (size_t)(first + t0 + tid) * p.heads + h;
-      keep[tid] = p.log_decay != nullptr ? expf(p.log_decay[at]) : fixed;
+      keep[tid] = p.log_decay != nullptr ? exp_of((A)p.log_decay[at]) : fixed;
       add[tid] = p.step != nullptr ? p.step[at] : p.k_scale;
     }
     __syncthreads();
     for (int t = 0; t < tokens; ++t) {
-      const float a = keep[t], value = vs[t][local], av = add[t] * value;
+      const A a = keep[t], value = vs[t][local], av = (A)add[t] * value;
       const float* kp = &ks[t][part * SEG];
       const float* qp = &qs[t][part * SEG];
-      float sum[4] = {0.f, 0.f, 0.f, 0.f};
+      A sum[4] = {0, 0, 0, 0};
 #pragma unroll
       for (int i = 0; i < PER; i += 4) {
         const float4 k4 = *(const float4*)(kp + i), q4 = *(const float4*)(qp + i);
-        s[i] = fmaf(a, s[i], k4.x * av);
-        s[i + 1] = fmaf(a, s[i + 1], k4.y * av);
-        s[i + 2] = fmaf(a, s[i + 2], k4.z * av);
-        s[i + 3] = fmaf(a, s[i + 3], k4.w * av);
-        sum[0] = fmaf(s[i], q4.x, sum[0]);
-        sum[1] = fmaf(s[i + 1], q4.y, sum[1]);
-        sum[2] = fmaf(s[i + 2], q4.z, sum[2]);
-        sum[3] = fmaf(s[i + 3], q4.w, sum[3]);
+        s[i] = fma(a, s[i], k4.x * av);
+        s[i + 1] = fma(a, s[i + 1], k4.y * av);
+        s[i + 2] = fma(a, s[i + 2], k4.z * av);
+        s[i + 3] = fma(a, s[i + 3], k4.w * av);
+        sum[0] = fma(s[i], (A)q4.x, sum[0]);
+        sum[1] = fma(s[i + 1], (A)q4.y, sum[1]);
+        sum[2] = fma(s[i + 2], (A)q4.z, sum[2]);
+        sum[3] = fma(s[i + 3], (A)q4.w, sum[3]);
       }
-      float total = (sum[0] + sum[1]) + (sum[2] + sum[3]);
+      A total = (sum[0] + sum[1]) + (sum[2] + sum[3]);
 #pragma unroll
       for (int o = WARP_COLS; o < 32; o <<= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
-      if (has_col && part == 0) p.o[((size_t)(first + t0 + t) * p.heads + h) * dv + col] = fmaf(skip, value, total);
+      if (has_col && part == 0) p.o[((size_t)(first + t0 + t) * p.heads + h) * dv + col] = (float)fma(skip, value, total);
     }
   }
   if (has_col) {
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
       const int row = part * PER + i;
-      if (row < n) st[(size_t)row * dv + col] = s[i];
+      if (row < n) st[(size_t)row * dv + col] = (float)s[i];
     }
   }
 }
@@ -166,9 +184,10 @@ constexpr int STEP_AHEAD = 8;          // 16-byte pieces of the state that a thr
 
 template <typename T, int CT>          // CT: value columns of a block
 __global__ void __launch_bounds__(STEP_THREADS) memory_step_kernel(const Memory p) {
+  using A = typename Carried<T>::type;
   constexpr int CG = CT / 4, LANES = STEP_THREADS / CG;
-  extern __shared__ float smem[];      // q [n], w k [n]
-  __shared__ float sums[STEP_THREADS / 32][CT];
+  extern __shared__ float smem[];      // q [n], k [n]
+  __shared__ A sums[STEP_THREADS / 32][CT];
   dependent_launch_trigger();
   const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * CT;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -188,20 +207,20 @@ __global__ void __launch_bounds__(STEP_THREADS) memory_step_kernel(const Memory 
   if (count != 1) return;
   const int g = h / (p.heads / p.groups);
   const size_t at = (size_t)first * p.heads + h;
-  const float w = p.step != nullptr ? p.step[at] : p.k_scale;
-  const float a = p.log_decay != nullptr ? expf(p.log_decay[at]) : p.head_decay[h];
+  const A w = p.step != nullptr ? p.step[at] : p.k_scale;
+  const A a = p.log_decay != nullptr ? exp_of((A)p.log_decay[at]) : (A)p.head_decay[h];
   float* qs = smem;
   float* ks = smem + n;
   for (int i = tid; i < n; i += STEP_THREADS) {
     qs[i] = to_float(((const T*)p.q)[(size_t)first * p.q_ld + g * n + i]);
-    ks[i] = w * to_float(((const T*)p.k)[(size_t)first * p.k_ld + g * n + i]);
+    ks[i] = to_float(((const T*)p.k)[(size_t)first * p.k_ld + g * n + i]);
   }
-  float v[4] = {0.f, 0.f, 0.f, 0.f};
+  A v[4] = {0, 0, 0, 0};               // the step times the value
   if (mine)
 #pragma unroll
-    for (int j = 0; j < 4; ++j) v[j] = to_float(((const T*)p.v)[(size_t)first * p.v_ld + h * dv + c + j]);
+    for (int j = 0; j < 4; ++j) v[j] = w * (A)to_float(((const T*)p.v)[(size_t)first * p.v_ld + h * dv + c + j]);
   __syncthreads();
-  float y[4] = {0.f, 0.f, 0.f, 0.f};
+  A y[4] = {0, 0, 0, 0};
   for (int base = 0; base < n; base += STEP_AHEAD * LANES) {
     if (base > 0) {
 #pragma unroll
@@ -214,16 +233,14 @@ __global__ void __launch_bounds__(STEP_THREADS) memory_step_kernel(const Memory 
     for (int i = 0; i < STEP_AHEAD; ++i) {
       const int row = base + r0 + i * LANES;
       if (!mine || row >= n) continue;
-      const float k = ks[row], q = qs[row];
-      s[i].x = fmaf(a, s[i].x, k * v[0]);
-      s[i].y = fmaf(a, s[i].y, k * v[1]);
-      s[i].z = fmaf(a, s[i].z, k * v[2]);
-      s[i].w = fmaf(a, s[i].w, k * v[3]);
-      *(float4*)(st + (size_t)row * dv + c) = s[i];
-      y[0] = fmaf(s[i].x, q, y[0]);
-      y[1] = fmaf(s[i].y, q, y[1]);
-      y[2] = fmaf(s[i].z, q, y[2]);
-      y[3] = fmaf(s[i].w, q, y[3]);
+      const A k = ks[row], q = qs[row];
+      const A s0 = fma(a, (A)s[i].x, k * v[0]), s1 = fma(a, (A)s[i].y, k * v[1]);
+      const A s2 = fma(a, (A)s[i].z, k * v[2]), s3 = fma(a, (A)s[i].w, k * v[3]);
+      *(float4*)(st + (size_t)row * dv + c) = make_float4((float)s0, (float)s1, (float)s2, (float)s3);
+      y[0] = fma(s0, q, y[0]);
+      y[1] = fma(s1, q, y[1]);
+      y[2] = fma(s2, q, y[2]);
+      y[3] = fma(s3, q, y[3]);
     }
   }
 #pragma unroll
@@ -235,11 +252,11 @@ __global__ void __launch_bounds__(STEP_THREADS) memory_step_kernel(const Memory 
     for (int j = 0; j < 4; ++j) sums[warp][lane * 4 + j] = y[j];
   __syncthreads();
   if (tid < CT && c0 + tid < dv) {
-    float total = 0.f;
+    A total = 0;
 #pragma unroll
     for (int i = 0; i < STEP_THREADS / 32; ++i) total += sums[i][tid];
-    if (p.skip != nullptr) total = fmaf(p.skip[h], to_float(((const T*)p.v)[(size_t)first * p.v_ld + h * dv + c0 + tid]), total);
-    p.o[at * dv + c0 + tid] = total;
+    if (p.skip != nullptr) total = fma((A)p.skip[h], (A)to_float(((const T*)p.v)[(size_t)first * p.v_ld + h * dv + c0 + tid]), total);
+    p.o[at * dv + c0 + tid] = (float)total;
   }
 }
 
