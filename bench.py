@@ -343,6 +343,44 @@ def finezen_config(size: dict, window: int = 1024, kv_rank: int = 512, experts: 
             "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": layers}
 
 
+def getozen_config(size: dict, head: int = 64, state: int = 128, groups: int = 4) -> dict:
+    """Getozen at the layer sizes of `size`: in turn a grouped-query attention (every earlier key, linearly
+    scaled frequencies, a gate per channel) beside a retention of half as many heads whose values are
+    twice as wide, and a Mamba-2 state space whose inner width is twice the model's (heads of `head`
+    channels, a state of `state`); every layer with a gated feed-forward of the dense width."""
+    d, width = size["dim"], size["width"]
+    mlp = {"kind": "dense", "ff": size["ff"]}
+    retained = size["heads"] // 2
+    parallel = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5,
+                 "rot": {"base": 10000.0, "dims": d, "scaling": {"factor": 4.0}}},
+        "right": {"heads": retained, "dim": d, "vdim": 2 * d, "decay": [1.0 - 2.0 ** (-5.0 - 5.0 * h / retained) for h in range(retained)],
+                  "rot": {"base": 10000.0, "dims": d}},
+        "left_scale": 1.0, "right_scale": 1.0}}
+    mamba = {"type": "mamba2", "mlp": mlp, "mixer": {"heads": 2 * width // head, "vdim": head, "state": state, "groups": groups, "conv": 4,
+                                                     "norm_groups": groups}}
+    layers = [json.loads(json.dumps((parallel, mamba)[i % 2])) for i in range(size["layers"])]
+    return {"architecture": "Getozen", "vocab": size["vocab"], "width": width, "norm": {"eps": 1e-6}, "layers": layers}
+
+
+def architectures_beside(only: str, size: dict) -> tuple:
+    """(name, configuration) of what `--only <name>` times at the layer sizes `size`: the architecture, the
+    closest of the others to it, and Qwen2."""
+    bidonex, qwen = bidonex_pair(size)
+    tail = (("qwen2", qwen),)
+    return {
+        "bidonex": (("bidonex", bidonex),),
+        # a float32 stream, windows, a recurrent layer
+        "zugarax": (("zugarax", zugarax_config(size)), ("bidonex", bidonex)),
+        # the same cached row per token and layer
+        "pukerax": (("pukerax", pukerax_config(size)), ("zugarax_latent", zugarax_latent_config(size))),
+        # a float32 stream, latent attention with a query latent and head gates, routed experts with a shared one
+        "finezen": (("finezen", finezen_config(size)), ("pukerax", pukerax_config(size))),
+        # a float32 stream, gated attention, a matrix-valued recurrent state, a dense gated feed-forward
+        "getozen": (("getozen", getozen_config(size)), ("zugarax", zugarax_config(size))),
+    }[only] + tail
+
+
 def step_cache_bytes(cache, contexts) -> float:
     """Cache bytes that a decode step reads: per page group the keys and values a request can see
     (all of its context, or the window and the kept first keys), and every recurrent state
@@ -357,27 +395,15 @@ def step_cache_bytes(cache, contexts) -> float:
     return total
 
 
-def bidonex_beside_qwen2(torch, peak: dict, steps: int, warmup: int, sizes, with_zugarax: bool = False, pukerax: bool = False,
-                         finezen: bool = False) -> dict:
-    """Prefill and decode of the architectures at equal layer sizes; `with_zugarax` puts Zugarax
-    in front of Bidonex (the closest of the others: a float32 stream, windows, a recurrent layer) and Qwen2;
-    `pukerax` times Pukerax beside Zugarax with latent attention in every layer (the closest to it) and Qwen2;
-    `finezen` times Finezen beside Pukerax (the closest to it: a float32 stream, latent attention with a query
-    latent and head gates, routed experts with a shared one) and Qwen2."""
+def beside_qwen2(torch, peak: dict, steps: int, warmup: int, sizes, only: str) -> dict:
+    """Prefill and decode of an architecture, of the closest of the others and of Qwen2 at equal layer sizes."""
     from paged_attention_engine_b200.engine.llm import Engine
     from paged_attention_engine_b200.sampling import SamplingRow
 
-    out: dict = {"only": "finezen" if finezen else "pukerax" if pukerax else "zugarax" if with_zugarax else "bidonex", "peaks": peak["source"], "sizes": {}}
+    out: dict = {"only": only, "peaks": peak["source"], "sizes": {}}
     for name in sizes:
-        bidonex, qwen = bidonex_pair(BIDONEX_SIZES[name])
         rows: dict = {}
-        archs = (("zugarax", zugarax_config(BIDONEX_SIZES[name])),) if with_zugarax else ()
-        archs = archs + (("bidonex", bidonex), ("qwen2", qwen))
-        if pukerax:
-            archs = (("pukerax", pukerax_config(BIDONEX_SIZES[name])), ("zugarax_latent", zugarax_latent_config(BIDONEX_SIZES[name])), ("qwen2", qwen))
-        if finezen:
-            archs = (("finezen", finezen_config(BIDONEX_SIZES[name])), ("pukerax", pukerax_config(BIDONEX_SIZES[name])), ("qwen2", qwen))
-        for arch, raw in archs:
+        for arch, raw in architectures_beside(only, BIDONEX_SIZES[name]):
             engine = Engine.from_random(raw, seed=0, dtype="bfloat16", device="cuda:0")
             row: dict = {"layers": BIDONEX_SIZES[name]["layers"], "weight_gb": round(engine.weight_bytes() / 1e9, 3)}
             for tokens in (512, 2048, 8192):
@@ -811,9 +837,9 @@ def main() -> int:
                         help="layer sizes for --only decode / prefill (the headline line is always the 1.5B shape)")
     parser.add_argument("--context", type=int, default=CONTEXT, help="context length for --only decode")
     parser.add_argument("--tokens", type=int, default=PREFILL_TOKENS, help="prompt length for --only prefill")
-    parser.add_argument("--arch", choices=("qwen2", "bidonex", "zugarax", "zugarax_latent", "pukerax", "finezen"), default="qwen2",
+    parser.add_argument("--arch", choices=("qwen2", "bidonex", "zugarax", "zugarax_latent", "pukerax", "finezen", "getozen"), default="qwen2",
                         help="with --only decode / prefill: the architecture that runs at the --shape's layer sizes")
-    parser.add_argument("--only", choices=("all", "decode", "prefill", "products", "stream7b", "pressure32b", "bidonex", "zugarax", "pukerax", "finezen"), default="all",
+    parser.add_argument("--only", choices=("all", "decode", "prefill", "products", "stream7b", "pressure32b", "bidonex", "zugarax", "pukerax", "finezen", "getozen"), default="all",
                         help="time one part only (for profiling); the JSON line then holds that part alone")
     args = parser.parse_args()
 
@@ -842,10 +868,9 @@ def main() -> int:
     if args.only == "pressure32b":
         print(json.dumps(pressure_32b(torch, args.layers_32b)))
         return 0
-    if args.only in ("bidonex", "zugarax", "pukerax", "finezen"):
+    if args.only in ("bidonex", "zugarax", "pukerax", "finezen", "getozen"):
         sizes = ("1.5b", "7b") if args.shape == "1.5b" else (args.shape,)
-        print(json.dumps(bidonex_beside_qwen2(torch, peak, args.steps, warmup, sizes, with_zugarax=args.only == "zugarax",
-                                              pukerax=args.only == "pukerax", finezen=args.only == "finezen")))
+        print(json.dumps(beside_qwen2(torch, peak, args.steps, warmup, sizes, args.only)))
         return 0
     if args.only == "products":
         for row in time_products({"1.5b": MODEL, "7b": MODEL_7B, "32b": MODEL_32B}[args.shape], args.batch, torch, peak):
@@ -865,7 +890,7 @@ def main() -> int:
             size["layers"] = args.layers
         args.layers = size["layers"]
         bidonex, model = bidonex_pair(size)
-        raw = {"zugarax": zugarax_config, "zugarax_latent": zugarax_latent_config, "pukerax": pukerax_config, "finezen": finezen_config}.get(args.arch, lambda size: bidonex)(size)
+        raw = {"zugarax": zugarax_config, "zugarax_latent": zugarax_latent_config, "pukerax": pukerax_config, "finezen": finezen_config, "getozen": getozen_config}.get(args.arch, lambda size: bidonex)(size)
         engine = Engine.from_random(raw, seed=0, dtype="bfloat16", device="cuda:0")
     else:
         engine = Engine.from_random(model, seed=0, dtype="bfloat16", device="cuda:0")

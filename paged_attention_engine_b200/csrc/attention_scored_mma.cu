@@ -292,17 +292,34 @@ __global__ void scored_merge_kernel(const ScoredParams p, int dv) {
       weights[s] = m == -FLT_MAX ? 0.f : fast_exp2(m - top);
     }
     __syncwarp();
-    if (lane == 0) {
-      float sum = sink2 != -FLT_MAX ? fast_exp2(sink2 - top) : 0.f;
-      for (int s = 0; s < p.splits; ++s) sum += p.part_sum[at + s] * weights[s];
-      stats[0] = sum > 0.f ? 1.f / sum : 0.f;
-    }
+    float sum = 0.f;
+    for (int s = lane; s < p.splits; s += 32) sum += p.part_sum[at + s] * weights[s];
+    sum = warp_sum(sum) + (sink2 != -FLT_MAX ? fast_exp2(sink2 - top) : 0.f);
+    if (lane == 0) stats[0] = sum > 0.f ? 1.f / sum : 0.f;
   }
   __syncthreads();
   const float inv = stats[0];
-  for (int c = threadIdx.x; c < dv; c += blockDim.x) {
-    float acc = 0.f;
-    for (int s = 0; s < p.splits; ++s) acc += p.part_out[(at + s) * dv + c] * weights[s];
+  // Every group of dv threads takes a share of the blocks' partial outputs, eight asked for at a time.
+  const int groups = blockDim.x / dv, group = threadIdx.x / dv, c = threadIdx.x - group * dv;
+  float acc = 0.f;
+  for (int s0 = group; s0 < p.splits; s0 += 8 * groups) {
+    float part[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int s = s0 + j * groups;
+      part[j] = s < p.splits ? p.part_out[(at + s) * dv + c] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int s = s0 + j * groups;
+      if (s < p.splits) acc = fmaf(part[j], weights[s], acc);
+    }
+  }
+  float* sums = weights + p.splits;            // [groups][dv]
+  sums[threadIdx.x] = acc;
+  __syncthreads();
+  if (group == 0) {
+    for (int g = 1; g < groups; ++g) acc += sums[g * dv + c];
     p.out[((size_t)first_token * p.heads + h) * dv + c] = __float2bfloat16_rn(acc * inv);
   }
 }
@@ -316,7 +333,7 @@ int launch(const ScoredParams& p, int seqs, int max_q_len, cudaStream_t s) {
   launch_kernel(scored_kernel<D, DV>, grid, 128, bytes, s, p);
   if (int err = check_launch("paged_attention_scored_mma")) return err;
   if (p.part_out != nullptr) {
-    launch_kernel(scored_merge_kernel, dim3(p.heads, seqs), 64, (size_t)p.splits * sizeof(float), s, p, DV);
+    launch_kernel(scored_merge_kernel, dim3(p.heads, seqs), 256, (size_t)(p.splits + 256) * sizeof(float), s, p, DV);
     return check_launch("paged_attention_scored_merge");
   }
   return 0;

@@ -35,6 +35,26 @@ struct DytStep {
   long long total;
 };
 
+// The planes of a split product added in their order, eight of them asked for at a time.
+__device__ __forceinline__ float plane_sum(const float* __restrict__ y, int planes, long long total, long long i) {
+  float s = y[i];
+  int k = 1;
+  for (; k + 8 <= planes; k += 8) {
+    float more[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) more[j] = y[(size_t)(k + j) * total + i];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s += more[j];
+  }
+  float rest[7];
+#pragma unroll
+  for (int j = 0; j < 7; ++j) rest[j] = k + j < planes ? y[(size_t)(k + j) * total + i] : 0.f;
+#pragma unroll
+  for (int j = 0; j < 7; ++j)
+    if (k + j < planes) s += rest[j];
+  return s;
+}
+
 template <typename TO>
 __global__ void __launch_bounds__(256) dyt_step_kernel(const DytStep p) {
   dependent_launch_prologue();
@@ -43,15 +63,12 @@ __global__ void __launch_bounds__(256) dyt_step_kernel(const DytStep p) {
   const int c = (int)(i % p.width);
   float v = p.x[i];
   if (p.y != nullptr) {
-    float s = p.y[i];
-    for (int k = 1; k < p.planes; ++k) s += p.y[(size_t)k * p.total + i];
+    float s = plane_sum(p.y, p.planes, p.total, i);
     if (p.post_w != nullptr) s = fmaf(tanhf(p.post_alpha[0] * s), p.post_w[c], p.post_b != nullptr ? p.post_b[c] : 0.f);
     v = fmaf(p.mult, s, v);
   }
   if (p.y2 != nullptr) {
-    float s = p.y2[i];
-    for (int k = 1; k < p.planes2; ++k) s += p.y2[(size_t)k * p.total + i];
-    v += s;
+    v += plane_sum(p.y2, p.planes2, p.total, i);
   }
   if (p.extra != nullptr) v += p.extra[i];
   if (p.x_new != nullptr) p.x_new[i] = v;
@@ -146,15 +163,17 @@ PAE_EXPORT int pae_dyt_step(float* x_new, void* normed, void* normed2, const flo
   cudaStream_t s = (cudaStream_t)stream;
   if (out_dtype != kF32 && out_dtype != kBF16) return fail(1, "dyt_step: unknown dtype %d", out_dtype);
   // The same operations per element either way: a token's numbers do not depend on which form ran.
-  if (width % 4 == 0 && aligned16(x) && aligned16(y) && aligned16(y2) && aligned16(extra) && aligned16(x_new) && aligned16(normed) && aligned16(normed2)) {
+  const bool few = total <= 64 * 1024;         // a column a thread, so that a decode step's few rows still fill some SMs
+  if (!few && width % 4 == 0 && aligned16(x) && aligned16(y) && aligned16(y2) && aligned16(extra) && aligned16(x_new) && aligned16(normed) && aligned16(normed2)) {
     const unsigned blocks = (unsigned)((total / 4 + 255) / 256);
     if (out_dtype == kF32) launch_kernel(dyt_step4_kernel<float>, blocks, 256, 0, s, p);
     else launch_kernel(dyt_step4_kernel<__nv_bfloat16>, blocks, 256, 0, s, p);
     return check_launch("dyt_step");
   }
-  const unsigned blocks = (unsigned)((total + 255) / 256);
-  if (out_dtype == kF32) launch_kernel(dyt_step_kernel<float>, blocks, 256, 0, s, p);
-  else launch_kernel(dyt_step_kernel<__nv_bfloat16>, blocks, 256, 0, s, p);
+  const int threads = few ? 64 : 256;
+  const unsigned blocks = (unsigned)((total + threads - 1) / threads);
+  if (out_dtype == kF32) launch_kernel(dyt_step_kernel<float>, blocks, threads, 0, s, p);
+  else launch_kernel(dyt_step_kernel<__nv_bfloat16>, blocks, threads, 0, s, p);
   return check_launch("dyt_step");
 }
 

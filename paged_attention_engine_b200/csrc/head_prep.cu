@@ -138,6 +138,66 @@ __global__ void __launch_bounds__(WARPS * 32) head_prep_kernel(const HeadPrep p)
   }
 }
 
+// The same without norms, for head sizes that split into pieces of 8 channels: a thread takes one piece
+// of one head of one token, either 8 neighbouring channels or, of a span whose pairs are half a span
+// apart, 4 channels and their 4 partners. No shared memory, 16-byte loads.
+__device__ __forceinline__ void store4(float* to, const float* v) { *(float4*)to = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(__nv_bfloat16* to, const float* v) {
+  uint2 packed;
+  *(__nv_bfloat162*)&packed.x = __floats2bfloat162_rn(v[0], v[1]);
+  *(__nv_bfloat162*)&packed.y = __floats2bfloat162_rn(v[2], v[3]);
+  *(uint2*)to = packed;
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(256) head_rotate_kernel(const HeadPrep p, long long total) {
+  dependent_launch_prologue();
+  const long long at = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (at >= total) return;
+  const int q_pieces = p.heads * (p.qd >> 3), k_pieces = p.kv_heads * (p.kd >> 3);
+  const int v_pieces = p.values != nullptr ? p.kv_heads * (p.dv >> 3) : 0;
+  const int per_token = q_pieces + k_pieces + v_pieces;
+  const int t = (int)(at / per_token);
+  int piece = (int)(at - (long long)t * per_token);
+  const bool is_q = piece < q_pieces, is_k = !is_q && piece < q_pieces + k_pieces;
+  piece -= is_q ? 0 : (is_k ? q_pieces : q_pieces + k_pieces);
+  const int d = is_q ? p.qd : (is_k ? p.kd : p.dv);
+  const int index = piece / (d >> 3), j = piece - index * (d >> 3);
+  TO* to;
+  if (is_q) {
+    to = (TO*)p.q_out + (size_t)t * p.q_ld + (size_t)index * d;
+  } else {
+    int slot = p.direct ? t : p.slots[t];
+    if (slot < 0 || (!p.direct && !slot_in_pool(slot, p.page_size))) return;
+    const int page = slot / p.page_size, offset = slot - page * p.page_size;
+    to = (TO*)(is_k ? p.keys : p.values) + (((size_t)page * p.kv_heads + index) * p.page_size + offset) * d;
+  }
+  const float* from = (const float*)p.proj + (size_t)t * p.ld + (is_q ? p.q_off : (is_k ? p.k_off : p.v_off)) + (size_t)index * d;
+  const bool turns = p.table != nullptr && (is_q || is_k) && j < (p.dims >> 3);
+  const int half = p.dims >> 1;
+  const int a = turns && !p.interleaved ? 4 * j : 8 * j, b = turns && !p.interleaved ? half + 4 * j : 8 * j + 4;
+  const float4 x4 = *(const float4*)(from + a), y4 = *(const float4*)(from + b);
+  float x[4] = {x4.x, x4.y, x4.z, x4.w}, y[4] = {y4.x, y4.y, y4.z, y4.w};
+  if (turns) {
+    const float* cs = p.table + (size_t)t * p.dims + 4 * j;
+    const float4 c4 = *(const float4*)cs, s4 = *(const float4*)(cs + half);
+    const float c[4] = {c4.x, c4.y, c4.z, c4.w}, s[4] = {s4.x, s4.y, s4.z, s4.w};
+    if (p.interleaved) {
+      rotate_pair(x[0], x[1], c[0], s[0]);
+      rotate_pair(x[2], x[3], c[1], s[1]);
+      rotate_pair(y[0], y[1], c[2], s[2]);
+      rotate_pair(y[2], y[3], c[3], s[3]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) rotate_pair(x[i], y[i], c[i], s[i]);
+    }
+  }
+  store4(to + a, x);
+  store4(to + b, y);
+}
+
+bool aligned16(const void* ptr) { return (((uintptr_t)ptr) & 15) == 0; }
+
 // table[t, i] = amplitude * cos(position[t] * inv_freq[i]), table[t, half + i] = amplitude * sin(same);
 // the angle is one float32 product.
 __global__ void rotary_table_amplitude_kernel(float* __restrict__ table, const int* __restrict__ positions,
@@ -214,6 +274,18 @@ PAE_EXPORT int pae_head_prep(void* q_out, int q_ld, void* keys, void* values, co
   HeadPrep p{proj, q_out, keys, values, q_norm, k_norm, table, slots, ld, q_ld, q_off, k_off, v_off, heads,
              slots != nullptr || direct ? kv_heads : 0, qd, kd, dv, q_span, k_span, q_rot0, k_rot0, table != nullptr ? dims : 0,
              interleaved, direct || page_size < 1 ? 1 : page_size, eps, whole, direct, kv_heads};
+  const int sizes = qd | (p.kv_heads > 0 ? kd | (values != nullptr ? dv : 0) : 0) | p.dims;
+  if (in_dtype == kF32 && q_norm == nullptr && k_norm == nullptr && q_rot0 == 0 && k_rot0 == 0 && sizes % 8 == 0 &&
+      ((ld | q_ld | q_off | k_off | v_off) & 3) == 0 && aligned16(proj) && aligned16(q_out) && aligned16(keys) && aligned16(values) &&
+      aligned16(table)) {
+    const long long total = (long long)tokens * (heads * (qd / 8) + p.kv_heads * (kd / 8 + (values != nullptr ? dv / 8 : 0)));
+    const int threads = total < 64 * 1024 ? 64 : 256;
+    const unsigned blocks = (unsigned)((total + threads - 1) / threads);
+    if (out_dtype == kF32) launch_kernel(head_rotate_kernel<float>, blocks, threads, 0, (cudaStream_t)stream, p, total);
+    else if (out_dtype == kBF16) launch_kernel(head_rotate_kernel<__nv_bfloat16>, blocks, threads, 0, (cudaStream_t)stream, p, total);
+    else return fail(1, "head_prep: element type %d is not supported", out_dtype);
+    return check_launch("head_prep");
+  }
   const int widest = qd > kd ? (qd > dv ? qd : dv) : (kd > dv ? kd : dv);
   const size_t smem = sizeof(float) * WARPS * (size_t)widest;
   if (smem > 48 * 1024) return fail(2, "head_prep: heads of %d channels are too wide", widest);

@@ -153,18 +153,27 @@ __global__ void __launch_bounds__(THREADS) ssm_prepare_kernel(const Prepare p) {
       for (int v = 0; v < VEC; ++v) w[j][v] = p.taps_w[(size_t)(c + v) * N + j];
 #pragma unroll
     for (int j = 0; j + 1 < N; ++j) window[j + 1] = raw(t0 - (N - 1) + j);
-    for (int t = 0; t < tokens; ++t) {
+    constexpr int AHEAD = 8;              // rows asked for at a time
+    for (int t1 = 0; t1 < tokens; t1 += AHEAD) {
+      Values<VEC> rows[AHEAD];
 #pragma unroll
-      for (int j = 0; j + 1 < N; ++j) window[j] = window[j + 1];
-      window[N - 1] = raw(t0 + t);
-      Values<VEC> acc = bias;
+      for (int i = 0; i < AHEAD; ++i)
+        if (t1 + i < tokens) rows[i] = projected<VEC>(p, (size_t)first + t0 + t1 + i, p.u_off + c);
 #pragma unroll
-      for (int j = 0; j < N; ++j)
+      for (int i = 0; i < AHEAD; ++i) {
+        if (t1 + i >= tokens) break;
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) acc.x[v] = fmaf(w[j][v], window[j].x[v], acc.x[v]);
+        for (int j = 0; j + 1 < N; ++j) window[j] = window[j + 1];
+        window[N - 1] = rows[i];
+        Values<VEC> acc = bias;
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) acc.x[v] = silu(acc.x[v]);
-      store<VEC>(out + (size_t)t * p.channels, acc);
+        for (int j = 0; j < N; ++j)
+#pragma unroll
+          for (int v = 0; v < VEC; ++v) acc.x[v] = fmaf(w[j][v], window[j].x[v], acc.x[v]);
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) acc.x[v] = silu(acc.x[v]);
+        store<VEC>(out + (size_t)(t1 + i) * p.channels, acc);
+      }
     }
   } else {
     for (int t = 0; t < tokens; ++t) {
@@ -219,7 +228,25 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) gated_group_norm_kernel(cons
   const float* y = p.y + token * p.groups * p.size + c0;
   const float* gate = p.gate + token * p.gate_ld + p.gate_off + c0;
   float squares = 0.f;
-  for (int i = lane * VEC; i < p.size; i += LANES * VEC) {
+  // the first KEPT pieces of a thread stay in registers, gated, all of them asked for at once
+  constexpr int KEPT = 8;
+  Values<VEC> ys[KEPT], gs[KEPT];
+#pragma unroll
+  for (int k = 0; k < KEPT; ++k) {
+    const int i = (lane + k * LANES) * VEC;
+    if (i < p.size) ys[k] = load<VEC>(y + i), gs[k] = load<VEC>(gate + i);
+  }
+#pragma unroll
+  for (int k = 0; k < KEPT; ++k) {
+    if ((lane + k * LANES) * VEC >= p.size) break;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      const float gated = ys[k].x[j] * silu(gs[k].x[j]), v = p.gate_first ? gated : ys[k].x[j];
+      squares = fmaf(v, v, squares);
+      ys[k].x[j] = gated;
+    }
+  }
+  for (int i = (lane + KEPT * LANES) * VEC; i < p.size; i += LANES * VEC) {
     Values<VEC> v = load<VEC>(y + i);
     if (p.gate_first) {
       const Values<VEC> g = load<VEC>(gate + i);
@@ -239,7 +266,18 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) gated_group_norm_kernel(cons
   }
   const float scale = p.mult / sqrtf(squares / (float)p.size + p.eps);
   T* out = (T*)p.out + token * p.out_ld + p.out_off + c0;
-  for (int i = lane * VEC; i < p.size; i += LANES * VEC) {
+#pragma unroll
+  for (int k = 0; k < KEPT; ++k) {
+    const int i = (lane + k * LANES) * VEC;
+    if (i >= p.size) break;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      ys[k].x[j] *= scale;
+      if (p.weight != nullptr) ys[k].x[j] *= p.weight[c0 + i + j];
+    }
+    store<VEC>(out + i, ys[k]);
+  }
+  for (int i = (lane + KEPT * LANES) * VEC; i < p.size; i += LANES * VEC) {
     Values<VEC> v = load<VEC>(y + i);
     const Values<VEC> g = load<VEC>(gate + i);
 #pragma unroll
@@ -253,7 +291,7 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) gated_group_norm_kernel(cons
 
 template <typename T, int VEC>
 void launch_group_norm(const GroupNorm& p, int tokens, cudaStream_t s) {
-  if (p.size > 512)
+  if (p.size > 1024)
     launch_kernel(gated_group_norm_kernel<T, VEC, true>, dim3(tokens, p.groups), 256, 0, s, p);
   else
     launch_kernel(gated_group_norm_kernel<T, VEC, false>, dim3(tokens, (p.groups + 3) / 4), 128, 0, s, p);

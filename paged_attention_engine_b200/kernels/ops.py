@@ -717,6 +717,12 @@ def _decode_attention(lib, out, qkv, keys, values, block_table, q_start, kv_len,
         _ptr(scratch), _stream()), launches)
 
 
+def plain_attention_takes(num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, dtype) -> bool:
+    """Whether `paged_attention` runs these sizes on its tensor-core kernels."""
+    return (dtype == torch.bfloat16 and use_tensor_cores
+            and bool(_lib("attention_mma").pae_attention_mma_supports(num_heads, num_kv_heads, head_dim, page_size)))
+
+
 def paged_attention(qkv, keys, values, block_table, q_start, q_pos0, kv_len, num_heads, num_kv_heads, head_dim,
                     page_size, max_q_len, max_kv_len, scale, window, num_single=None, form: int = 0,
                     info: dict | None = None, multi_index: torch.Tensor | None = None) -> torch.Tensor:

@@ -112,11 +112,19 @@ class GatedWindowAttention(ProjectedMixer):
         group = ctx.groups[cache.group]
         h, g, d, dv = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim
         table = self.position_encoding.table(ctx) if self.position_encoding is not None else None
+        # A rule without a sink over heads of one size is what the plain attention kernels compute; they
+        # take the queries as the leading columns of q|k|v rows.
+        plain = self.sink is None and d == dv and ops.plain_attention_takes(h, g, d, cache.page_size, self.runtime.dtype)
+        q_rows = torch.empty((proj.shape[0], (h + 2 * g) * d), dtype=self.runtime.dtype, device=proj.device) if plain else None
         q = ops.head_prep(
             proj, q_off=offset, k_off=offset + h * d, v_off=offset + (h + g) * d, heads=h, kv_heads=g, q_dim=d, k_dim=d, value_dim=dv,
             q_norm=self.q_norm, k_norm=self.k_norm, q_span=d, k_span=d, eps=float(self.norm_eps or 0.0),
             table=table, interleaved=self.interleaved, q_rot0=0, k_rot0=0, slots=group.slots if cache.writes else None,
-            keys=cache.keys, values=cache.values, page_size=cache.page_size, out_dtype=self.runtime.dtype, whole=self.whole_norm)
+            keys=cache.keys, values=cache.values, page_size=cache.page_size, out_dtype=self.runtime.dtype, whole=self.whole_norm, q_out=q_rows)
+        if plain:
+            return ops.paged_attention(
+                q, cache.keys, cache.values, group.block_table, ctx.q_start, ctx.q_pos0, ctx.kv_len, h, g, d, cache.page_size,
+                ctx.max_q_len, ctx.max_kv_len, self.scale, self.window, num_single=ctx.num_single, multi_index=ctx.multi_index)
         return ops.paged_attention_scored(
             q, cache.keys, cache.values, group.block_table, ctx.q_start, ctx.q_pos0, ctx.kv_len, h, g, d, dv,
             cache.page_size, ctx.max_q_len, self.scale, sink=self.sink, window=self.window,
