@@ -316,7 +316,7 @@ __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint3
   lo = pack_bf16(a - back.x, b - back.y);
 }
 
-// One chunk's own contribution to the state: a 64 x 64 tile of U per block, a warp 16 key channels.
+// One chunk's own contribution to the state: a 64 x 64 tile of U per block, a warp 32 x 32 of it.
 constexpr int ST_PITCH = 72;            // bfloat16 elements between rows of a 64-wide tile
 __global__ void __launch_bounds__(128) memory_chunk_states_kernel(const Memory p) {
   dependent_launch_prologue();
@@ -370,43 +370,60 @@ __global__ void __launch_bounds__(128) memory_chunk_states_kernel(const Memory p
   }
   cp_async_wait<0>();
   __syncthreads();
-  if (n0 + warp * 16 >= p.n) return;
+  const int wn = (warp & 1) * 32, wd = (warp >> 1) * 32;       // the warp's corner of the tile
+  if (n0 + wn >= p.n || d0 + wd >= p.dv) return;
   const int mid = lane >> 3, r = lane & 7;
-  float acc[8][4];
+  float acc[2][4][4];
 #pragma unroll
-  for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
   const int steps = (count + 15) / 16;
+#pragma unroll 2
   for (int t = 0; t < steps; ++t) {
-    uint32_t a[4];                       // rows: key channels, columns: tokens
-    ldmatrix_x4_trans(a, smem_u32(ks + (t * 16 + (mid >> 1) * 8 + r) * ST_PITCH + warp * 16 + (mid & 1) * 8));
+    uint32_t a[2][4], hi[2][4], lo[2][4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int at = (t * 16 + (mid & 1) * 8 + r) * ST_PITCH + j * 16 + (mid >> 1) * 8;
-      uint32_t hi[4], lo[4];
-      ldmatrix_x4_trans(hi, smem_u32(vh + at));
-      ldmatrix_x4_trans(lo, smem_u32(vl + at));
-      mma_16816(acc[2 * j], a, hi[0], hi[1]);
-      mma_16816(acc[2 * j + 1], a, hi[2], hi[3]);
-      mma_16816(acc[2 * j], a, lo[0], lo[1]);
-      mma_16816(acc[2 * j + 1], a, lo[2], lo[3]);
+    for (int m = 0; m < 2; ++m)          // rows: key channels, columns: tokens
+      ldmatrix_x4_trans(a[m], smem_u32(ks + (t * 16 + (mid >> 1) * 8 + r) * ST_PITCH + wn + m * 16 + (mid & 1) * 8));
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int at = (t * 16 + (mid & 1) * 8 + r) * ST_PITCH + wd + j * 16 + (mid >> 1) * 8;
+      ldmatrix_x4_trans(hi[j], smem_u32(vh + at));
+      ldmatrix_x4_trans(lo[j], smem_u32(vl + at));
     }
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        mma_16816(acc[m][2 * j], a[m], hi[j][0], hi[j][1]);
+        mma_16816(acc[m][2 * j + 1], a[m], hi[j][2], hi[j][3]);
+      }
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        mma_16816(acc[m][2 * j], a[m], lo[j][0], lo[j][1]);
+        mma_16816(acc[m][2 * j + 1], a[m], lo[j][2], lo[j][3]);
+      }
   }
   float* out = p.chunk_state + ((size_t)chunk_slot(first, i, chunk) * p.heads + h) * p.n * p.dv;
 #pragma unroll
-  for (int half = 0; half < 2; ++half) {
-    const int row = n0 + warp * 16 + (lane >> 2) + half * 8;
-    if (row >= p.n) continue;
+  for (int m = 0; m < 2; ++m)
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int col = d0 + j * 8 + (lane & 3) * 2;
-      if (col < p.dv) *(float2*)(out + (size_t)row * p.dv + col) = make_float2(acc[j][half * 2], acc[j][half * 2 + 1]);
+    for (int half = 0; half < 2; ++half) {
+      const int row = n0 + wn + m * 16 + (lane >> 2) + half * 8;
+      if (row >= p.n) continue;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int col = d0 + wd + j * 8 + (lane & 3) * 2;
+        if (col < p.dv) *(float2*)(out + (size_t)row * p.dv + col) = make_float2(acc[m][j][half * 2], acc[m][j][half * 2 + 1]);
+      }
     }
-  }
 }
 
 // From chunk to chunk: the state before each (as two bfloat16 planes), and the new state. Four
 // neighbouring elements a thread; the contributions of PASS_AHEAD chunks are in flight at a time.
-constexpr int PASS_AHEAD = 4;
+constexpr int PASS_AHEAD = 8;
 __global__ void __launch_bounds__(256) memory_chunk_pass_kernel(const Memory p) {
   dependent_launch_prologue();
   const int h = blockIdx.y, i = blockIdx.z, b = p.list != nullptr ? p.list[i] : i;
@@ -516,18 +533,18 @@ __global__ void __launch_bounds__(256) memory_chunk_output_kernel(const Memory p
   const uint32_t q_at = smem_u32(qs + (size_t)(row0 + (mid & 1) * 8 + r) * kp + (mid >> 1) * 8);
   if (live) {
     for (int t = 0; t < np / 16; ++t) {
-      uint32_t a[4];
+      uint32_t a[4], s4[DVT / 16][4];
       ldmatrix_x4(a, q_at + t * 32);
 #pragma unroll
-      for (int j = 0; j < DVT / 16; ++j) {
-        const int at = (t * 16 + (mid & 1) * 8 + r) * VP + j * 16 + (mid >> 1) * 8;
-        uint32_t hi[4], lo[4];
-        ldmatrix_x4_trans(hi, smem_u32(sh + at));
-        ldmatrix_x4_trans(lo, smem_u32(sl + at));
-        mma_16816(acc[2 * j], a, hi[0], hi[1]);
-        mma_16816(acc[2 * j + 1], a, hi[2], hi[3]);
-        mma_16816(acc[2 * j], a, lo[0], lo[1]);
-        mma_16816(acc[2 * j + 1], a, lo[2], lo[3]);
+      for (int plane = 0; plane < 2; ++plane) {
+        const __nv_bfloat16* from = (plane == 0 ? sh : sl) + (t * 16 + (mid & 1) * 8 + r) * VP + (mid >> 1) * 8;
+#pragma unroll
+        for (int j = 0; j < DVT / 16; ++j) ldmatrix_x4_trans(s4[j], smem_u32(from + j * 16));
+#pragma unroll
+        for (int j = 0; j < DVT / 16; ++j) {
+          mma_16816(acc[2 * j], a, s4[j][0], s4[j][1]);
+          mma_16816(acc[2 * j + 1], a, s4[j][2], s4[j][3]);
+        }
       }
     }
   }
@@ -554,36 +571,49 @@ __global__ void __launch_bounds__(256) memory_chunk_output_kernel(const Memory p
     const __nv_bfloat16* kt = half == 0 ? k0 : k1;
     const __nv_bfloat16* vt = half == 0 ? v0 : v1;
     const int blocks = row0 >= half * 64 + 64 ? 4 : (row0 - half * 64) / 16 + 1;      // 16-token steps that the warp's rows see
-    for (int u = 0; u < blocks; ++u) {
-      float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-      const uint32_t k_at = smem_u32(kt + (size_t)(u * 16 + (mid >> 1) * 8 + r) * kp + (mid & 1) * 8);
+    for (int u0 = 0; u0 < blocks; u0 += 2) {           // two of them at a time (the second may be beyond the rows: all masked)
+      float s[4][4];
+#pragma unroll
+      for (int w = 0; w < 4; ++w) s[w][0] = s[w][1] = s[w][2] = s[w][3] = 0.f;
+      const uint32_t k_at = smem_u32(kt + (size_t)(u0 * 16 + (mid >> 1) * 8 + r) * kp + (mid & 1) * 8);
+      const uint32_t k_next = k_at + 16 * kp * 2;
+#pragma unroll 4
       for (int t = 0; t < np / 16; ++t) {
-        uint32_t a[4], k4[4];
+        uint32_t a[4], ka[4], kb[4];
         ldmatrix_x4(a, q_at + t * 32);
-        ldmatrix_x4(k4, k_at + t * 32);
-        mma_16816(s[0], a, k4[0], k4[1]);
-        mma_16816(s[1], a, k4[2], k4[3]);
+        ldmatrix_x4(ka, k_at + t * 32);
+        ldmatrix_x4(kb, k_next + t * 32);
+        mma_16816(s[0], a, ka[0], ka[1]);
+        mma_16816(s[1], a, ka[2], ka[3]);
+        mma_16816(s[2], a, kb[0], kb[1]);
+        mma_16816(s[3], a, kb[2], kb[3]);
       }
 #pragma unroll
-      for (int w = 0; w < 2; ++w)
+      for (int w = 0; w < 4; ++w)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int row = my_row[e >> 1], token = half * 64 + u * 16 + w * 8 + (lane & 3) * 2 + (e & 1);
-          s[w][e] = token <= row ? s[w][e] * (weight[token] * exp2f(my_cumulative[e >> 1] - cumulative[token])) : 0.f;
+          const int row = my_row[e >> 1], token = half * 64 + u0 * 16 + w * 8 + (lane & 3) * 2 + (e & 1);
+          s[w][e] = token <= row ? s[w][e] * (weight[token] * fast_exp2(my_cumulative[e >> 1] - cumulative[token])) : 0.f;
         }
-      uint32_t hi[4], lo[4];
-      split_pair(s[0][0], s[0][1], hi[0], lo[0]);
-      split_pair(s[0][2], s[0][3], hi[1], lo[1]);
-      split_pair(s[1][0], s[1][1], hi[2], lo[2]);
-      split_pair(s[1][2], s[1][3], hi[3], lo[3]);
 #pragma unroll
-      for (int j = 0; j < DVT / 16; ++j) {
-        uint32_t v4[4];
-        ldmatrix_x4_trans(v4, smem_u32(vt + (size_t)(u * 16 + (mid & 1) * 8 + r) * VP + j * 16 + (mid >> 1) * 8));
-        mma_16816(acc[2 * j], hi, v4[0], v4[1]);
-        mma_16816(acc[2 * j + 1], hi, v4[2], v4[3]);
-        mma_16816(acc[2 * j], lo, v4[0], v4[1]);
-        mma_16816(acc[2 * j + 1], lo, v4[2], v4[3]);
+      for (int x = 0; x < 2; ++x) {
+        if (u0 + x >= blocks) break;
+        uint32_t hi[4], lo[4], v4[DVT / 16][4];
+#pragma unroll
+        for (int j = 0; j < DVT / 16; ++j)
+          ldmatrix_x4_trans(v4[j], smem_u32(vt + (size_t)((u0 + x) * 16 + (mid & 1) * 8 + r) * VP + j * 16 + (mid >> 1) * 8));
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split_pair(s[2 * x + (e >> 1)][(e & 1) * 2], s[2 * x + (e >> 1)][(e & 1) * 2 + 1], hi[e], lo[e]);
+#pragma unroll
+        for (int j = 0; j < DVT / 16; ++j) {
+          mma_16816(acc[2 * j], hi, v4[j][0], v4[j][1]);
+          mma_16816(acc[2 * j + 1], hi, v4[j][2], v4[j][3]);
+        }
+#pragma unroll
+        for (int j = 0; j < DVT / 16; ++j) {
+          mma_16816(acc[2 * j], lo, v4[j][0], v4[j][1]);
+          mma_16816(acc[2 * j + 1], lo, v4[j][2], v4[j][3]);
+        }
       }
     }
   }

@@ -16,8 +16,9 @@ import torch
 
 F = torch.float64
 
-# A function applied to every sublayer's input (the normed stream), or None. Tests set it to a
-# rounding to bfloat16 to learn how far one rounding of an input moves a model's logits.
+# A function applied wherever a 16-bit engine hands numbers on as 16 bits (a sublayer's input, heads
+# after rotation, channels after the convolution, an output product's operand), or None. Tests set it to
+# a rounding to bfloat16 to learn how far such roundings move a model's logits.
 narrow = None
 
 
@@ -25,7 +26,7 @@ def _f(t):
     return t.to(F)
 
 
-def _input(h):
+def _handed(h):
     return narrow(h) if narrow is not None else h
 
 
@@ -92,9 +93,9 @@ def attention_mixer(h, tensors, name, m):
     biased = lambda n: proj(n) + _f(tensors[f"{name}.{n}.b"])
     q, k, v = (biased(n).view(T, heads, size) for n, heads, size in
                (("q", m["heads"], m["dim"]), ("k", m["kv_heads"], m["dim"]), ("v", m["kv_heads"], m["vdim"])))
-    o = causal_attention(rotate(q, m["rot"], True), rotate(k, m["rot"], True), v, m["scale"])
+    o = _handed(causal_attention(_handed(rotate(q, m["rot"], True)), _handed(rotate(k, m["rot"], True)), _handed(v), m["scale"]))
     gate = 1.0 / (1.0 + torch.exp(-proj("g")))
-    return (o.reshape(T, -1) * gate) @ _f(tensors[f"{name}.o"]).T
+    return _handed(o.reshape(T, -1) * gate) @ _f(tensors[f"{name}.o"]).T
 
 
 # --------------------------------------------------------------------------- #
@@ -116,11 +117,11 @@ def decayed_memory(q, k, v, keep, state=None):
 def retention_mixer(h, tensors, name, m, eps):
     T, H = h.shape[0], m["heads"]
     proj = lambda n: h @ _f(tensors[f"{name}.{n}"]).T
-    q, k = rotate(proj("q").view(T, H, -1), m["rot"], False), rotate(proj("k").view(T, H, -1), m["rot"], False)
+    q, k = (_handed(rotate(proj(n).view(T, H, -1), m["rot"], False)) for n in ("q", "k"))
     k = k * float(m["dim"]) ** -0.5
     keep = torch.tensor(m["decay"], dtype=F).expand(T, H)
-    o, _ = decayed_memory(q, k, proj("v").view(T, H, -1), keep)
-    return (unit_rms(o, eps).reshape(T, -1) * silu(proj("g"))) @ _f(tensors[f"{name}.o"]).T
+    o, _ = decayed_memory(q, k, _handed(proj("v").view(T, H, -1)), keep)
+    return _handed(unit_rms(o, eps).reshape(T, -1) * silu(proj("g"))) @ _f(tensors[f"{name}.o"]).T
 
 
 def short_convolution(u, taps, bias):
@@ -143,13 +144,13 @@ def mamba2_mixer(h, tensors, name, m, eps):
     T, H, dv, n, G = h.shape[0], m["heads"], m["vdim"], m["state"], m["groups"]
     inner = H * dv
     z, xbc, dt = (h @ _f(tensors[f"{name}.in"]).T).split([inner, inner + 2 * G * n, H], dim=1)
-    xbc = silu(short_convolution(xbc, tensors[f"{name}.conv"], tensors[f"{name}.conv.b"]))
+    xbc = _handed(silu(short_convolution(xbc, tensors[f"{name}.conv"], tensors[f"{name}.conv.b"])))
     x, B, C = xbc.split([inner, G * n, G * n], dim=1)
     step = softplus(dt + _f(tensors[f"{name}.dt_bias"]))
     y = selective_memory(x.view(T, H, dv), B.view(T, G, n), C.view(T, G, n), step, torch.exp(_f(tensors[f"{name}.A_log"])),
                          _f(tensors[f"{name}.D"])).reshape(T, inner)
     y = unit_rms((y * silu(z)).view(T, m["norm_groups"], -1), eps).reshape(T, inner) * _f(tensors[f"{name}.norm"])
-    return y @ _f(tensors[f"{name}.o"]).T
+    return _handed(y) @ _f(tensors[f"{name}.o"]).T
 
 
 # --------------------------------------------------------------------------- #
@@ -165,14 +166,14 @@ def mixer(h, tensors, name, kind, m, eps):
 
 def relu_glu(h, tensors, name):
     gate, up = h @ _f(tensors[f"{name}.gate"]).T, h @ _f(tensors[f"{name}.up"]).T
-    return (torch.maximum(gate, torch.zeros_like(gate)) * up) @ _f(tensors[f"{name}.down"]).T
+    return _handed(torch.maximum(gate, torch.zeros_like(gate)) * up) @ _f(tensors[f"{name}.down"]).T
 
 
 def layer(x, tensors, name, entry, eps):
     """Both sublayers read the same x, each through a norm of its own."""
-    out = mixer(_input(dynamic_tanh(x, tensors, f"{name}.norm1")), tensors, f"{name}.mix", entry["type"], entry["mixer"], eps)
+    out = mixer(_handed(dynamic_tanh(x, tensors, f"{name}.norm1")), tensors, f"{name}.mix", entry["type"], entry["mixer"], eps)
     if entry.get("mlp"):
-        out = out + relu_glu(_input(dynamic_tanh(x, tensors, f"{name}.norm2")), tensors, f"{name}.mlp")
+        out = out + relu_glu(_handed(dynamic_tanh(x, tensors, f"{name}.norm2")), tensors, f"{name}.mlp")
     return x + out
 
 
