@@ -316,48 +316,57 @@ __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint3
   lo = pack_bf16(a - back.x, b - back.y);
 }
 
-// One chunk's own contribution to the state: a 64 x 64 tile of U per block, a warp 32 x 32 of it.
+// One chunk's own contribution to the state: an NT x 64 tile of U per block, a warp 32 x 32 of it (NT 64 or 128
+// key channels: the weighted values are split once for all of them).
 constexpr int ST_PITCH = 72;            // bfloat16 elements between rows of a 64-wide tile
-__global__ void __launch_bounds__(128) memory_chunk_states_kernel(const Memory p) {
+template <int NT>
+__host__ __device__ constexpr size_t states_smem() { return 2 * (size_t)CHUNK * (NT + 8 + 2 * ST_PITCH); }
+
+template <int NT>
+__global__ void __launch_bounds__(2 * NT) memory_chunk_states_kernel(const Memory p) {
   dependent_launch_prologue();
+  constexpr int THREADS = 2 * NT, K_PITCH = NT + 8, K_PIECES = NT / 8, V_PER = CHUNK * 8 / THREADS;
   extern __shared__ __align__(16) unsigned char raw[];
   __shared__ float cumulative[CHUNK], weight[CHUNK];
-  const int n_tiles = (p.n + 63) / 64, dv_tiles = (p.dv + 63) / 64;
+  const int n_tiles = (p.n + NT - 1) / NT, dv_tiles = (p.dv + 63) / 64;
   const int tile = blockIdx.x % (n_tiles * dv_tiles), chunk = blockIdx.x / (n_tiles * dv_tiles);
   const int h = blockIdx.y, i = blockIdx.z, b = p.list != nullptr ? p.list[i] : i;
   const int first = p.q_start[b], all = p.q_start[b + 1] - first;
   const int count = min(CHUNK, all - chunk * CHUNK);
   if (all == 1 || count <= 0) return;
-  const int n0 = (tile % n_tiles) * 64, d0 = (tile / n_tiles) * 64;
+  const int n0 = (tile % n_tiles) * NT, d0 = (tile / n_tiles) * 64;
   const int g = h / (p.heads / p.groups);
   const size_t token0 = (size_t)first + chunk * CHUNK;
-  __nv_bfloat16* ks = (__nv_bfloat16*)raw;                  // [CHUNK][ST_PITCH]
-  __nv_bfloat16* vh = ks + CHUNK * ST_PITCH;
+  __nv_bfloat16* ks = (__nv_bfloat16*)raw;                  // [CHUNK][K_PITCH]
+  __nv_bfloat16* vh = ks + CHUNK * K_PITCH;                 // [CHUNK][ST_PITCH]
   __nv_bfloat16* vl = vh + CHUNK * ST_PITCH;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  for (int e = tid; e < CHUNK * 8; e += 128) {
-    const int row = e >> 3, ch = (e & 7) * 8;
-    __nv_bfloat16* to = ks + row * ST_PITCH + ch;
+#pragma unroll
+  for (int e = tid; e < CHUNK * K_PIECES; e += THREADS) {
+    const int row = e / K_PIECES, ch = (e % K_PIECES) * 8;
+    __nv_bfloat16* to = ks + row * K_PITCH + ch;
     if (row < count && n0 + ch < p.n)
       cp_async16(smem_u32(to), (const __nv_bfloat16*)p.k + (token0 + row) * p.k_ld + g * p.n + n0 + ch);
     else
       *(uint4*)to = make_uint4(0, 0, 0, 0);
   }
   cp_async_commit();
-  uint4 raw_v[8];
+  uint4 raw_v[V_PER];
 #pragma unroll
-  for (int j = 0; j < 8; ++j) {
-    const int e = tid + j * 128, row = e >> 3, ch = (e & 7) * 8;
+  for (int j = 0; j < V_PER; ++j) {
+    const int e = tid + j * THREADS, row = e >> 3, ch = (e & 7) * 8;
     raw_v[j] = row < count && d0 + ch < p.dv ? *(const uint4*)((const __nv_bfloat16*)p.v + (token0 + row) * p.v_ld + h * p.dv + d0 + ch)
                                              : make_uint4(0, 0, 0, 0);
   }
   chunk_decays(p, token0, count, h, cumulative, weight);
   const float last = cumulative[CHUNK - 1];
   if (tile == 0 && tid == 0) p.chunk_decay[(size_t)chunk_slot(first, i, chunk) * p.heads + h] = exp2f(last);
+  if (tid < CHUNK) weight[tid] *= exp2f(last - cumulative[tid]);
+  __syncthreads();
 #pragma unroll
-  for (int j = 0; j < 8; ++j) {
-    const int e = tid + j * 128, row = e >> 3, ch = (e & 7) * 8;
-    const float w = weight[row] * exp2f(last - cumulative[row]);
+  for (int j = 0; j < V_PER; ++j) {
+    const int e = tid + j * THREADS, row = e >> 3, ch = (e & 7) * 8;
+    const float w = weight[row];
     const __nv_bfloat162* v2 = (const __nv_bfloat162*)&raw_v[j];
     uint32_t hi[4], lo[4];
 #pragma unroll
@@ -370,7 +379,7 @@ __global__ void __launch_bounds__(128) memory_chunk_states_kernel(const Memory p
   }
   cp_async_wait<0>();
   __syncthreads();
-  const int wn = (warp & 1) * 32, wd = (warp >> 1) * 32;       // the warp's corner of the tile
+  const int wn = (warp >> 1) * 32, wd = (warp & 1) * 32;       // the warp's corner of the tile
   if (n0 + wn >= p.n || d0 + wd >= p.dv) return;
   const int mid = lane >> 3, r = lane & 7;
   float acc[2][4][4];
@@ -384,7 +393,7 @@ __global__ void __launch_bounds__(128) memory_chunk_states_kernel(const Memory p
     uint32_t a[2][4], hi[2][4], lo[2][4];
 #pragma unroll
     for (int m = 0; m < 2; ++m)          // rows: key channels, columns: tokens
-      ldmatrix_x4_trans(a[m], smem_u32(ks + (t * 16 + (mid >> 1) * 8 + r) * ST_PITCH + wn + m * 16 + (mid & 1) * 8));
+      ldmatrix_x4_trans(a[m], smem_u32(ks + (t * 16 + (mid >> 1) * 8 + r) * K_PITCH + wn + m * 16 + (mid & 1) * 8));
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int at = (t * 16 + (mid & 1) * 8 + r) * ST_PITCH + wd + j * 16 + (mid >> 1) * 8;
@@ -478,7 +487,7 @@ template <int DVT>
 __global__ void __launch_bounds__(256) memory_chunk_output_kernel(const Memory p) {
   dependent_launch_prologue();
   extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ float cumulative[CHUNK], weight[CHUNK];
+  __shared__ __align__(16) float cumulative[CHUNK], weight[CHUNK];
   const int dv_tiles = (p.dv + DVT - 1) / DVT;
   const int d0 = (blockIdx.x % dv_tiles) * DVT, chunk = blockIdx.x / dv_tiles;
   const int h = blockIdx.y, i = blockIdx.z, b = p.list != nullptr ? p.list[i] : i;
@@ -499,14 +508,21 @@ __global__ void __launch_bounds__(256) memory_chunk_output_kernel(const Memory p
   __nv_bfloat16* v1 = k1 + (size_t)64 * kp;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   auto fetch_rows = [&](__nv_bfloat16* to, int pitch, const __nv_bfloat16* from, size_t ld, int rows, int limit, int cols, int valid_cols) {
-    const int chunks = cols >> 3;
-    for (int e = tid; e < rows * chunks; e += 256) {
-      const int row = e / chunks, c = (e - row * chunks) * 8;
-      __nv_bfloat16* at = to + (size_t)row * pitch + c;
-      if (row < limit && c < valid_cols)
-        cp_async16(smem_u32(at), from + (size_t)row * ld + c);
+    // a thread keeps its column and steps through the rows (cols <= 2048)
+    const int chunks = cols >> 3, stride = 256 / chunks, first_row = tid / chunks, c = (tid - first_row * chunks) * 8;
+    if (first_row >= stride) return;
+    const bool valid = c < valid_cols;
+    __nv_bfloat16* at = to + first_row * pitch + c;
+    const __nv_bfloat16* src = from + first_row * ld + c;
+    const size_t src_step = stride * ld;
+#pragma unroll 4
+    for (int row = first_row; row < rows; row += stride) {
+      if (valid && row < limit)
+        cp_async16(smem_u32(at), src);
       else
         *(uint4*)at = make_uint4(0, 0, 0, 0);
+      at += stride * pitch;
+      src += src_step;
     }
   };
   const __nv_bfloat16* q_from = (const __nv_bfloat16*)p.q + token0 * p.q_ld + g * n;
@@ -589,12 +605,15 @@ __global__ void __launch_bounds__(256) memory_chunk_output_kernel(const Memory p
         mma_16816(s[3], a, kb[2], kb[3]);
       }
 #pragma unroll
-      for (int w = 0; w < 4; ++w)
+      for (int w = 0; w < 4; ++w) {
+        const int token = half * 64 + u0 * 16 + w * 8 + (lane & 3) * 2;
+        const float2 c2 = *(const float2*)(cumulative + token), w2 = *(const float2*)(weight + token);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int row = my_row[e >> 1], token = half * 64 + u0 * 16 + w * 8 + (lane & 3) * 2 + (e & 1);
-          s[w][e] = token <= row ? s[w][e] * (weight[token] * fast_exp2(my_cumulative[e >> 1] - cumulative[token])) : 0.f;
+          const float c = e & 1 ? c2.y : c2.x, wt = e & 1 ? w2.y : w2.x;
+          s[w][e] = token + (e & 1) <= my_row[e >> 1] ? s[w][e] * (wt * fast_exp2(my_cumulative[e >> 1] - c)) : 0.f;
         }
+      }
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         if (u0 + x >= blocks) break;
@@ -728,9 +747,13 @@ PAE_EXPORT int pae_decay_memory_chunked(float* o, float* state, long long slot_s
     return fail(2, "decay_memory_chunked: an operand does not start on a 16-byte boundary");
   cudaStream_t s = (cudaStream_t)stream;
   const int chunks = (max_q_len + CHUNK - 1) / CHUNK;
-  const size_t states_smem = (size_t)3 * CHUNK * ST_PITCH * 2;
-  if (int err = allow_smem(memory_chunk_states_kernel, states_smem, "decay_memory_chunked")) return err;
-  launch_kernel(memory_chunk_states_kernel, dim3(chunks * ((n + 63) / 64) * ((dv + 63) / 64), heads, listed), 128, states_smem, s, p);
+  if (n > 64) {
+    if (int err = allow_smem(memory_chunk_states_kernel<128>, states_smem<128>(), "decay_memory_chunked")) return err;
+    launch_kernel(memory_chunk_states_kernel<128>, dim3(chunks * ((n + 127) / 128) * ((dv + 63) / 64), heads, listed), 256, states_smem<128>(), s, p);
+  } else {
+    if (int err = allow_smem(memory_chunk_states_kernel<64>, states_smem<64>(), "decay_memory_chunked")) return err;
+    launch_kernel(memory_chunk_states_kernel<64>, dim3(chunks * ((dv + 63) / 64), heads, listed), 128, states_smem<64>(), s, p);
+  }
   if (int err = check_launch("decay_memory_chunk_states")) return err;
   launch_kernel(memory_chunk_pass_kernel, dim3((unsigned)(((size_t)n * dv / 4 + 255) / 256), heads, listed), 256, 0, s, p);
   if (int err = check_launch("decay_memory_chunk_pass")) return err;

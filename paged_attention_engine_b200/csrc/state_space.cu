@@ -40,7 +40,7 @@ struct Prepare {
   const int* state_slot;
   long long slot_stride, plane;
   int planes, ld, z_off, z_cols, u_off, channels, dt_off, heads, taps;
-  int u_blocks, z_blocks;   // blockIdx.x: channels of u, then of z, then heads
+  int u_blocks, z_blocks;   // blockIdx.x: channels of u, then of z, then heads of the block's tokens
 };
 
 template <int VEC>
@@ -80,7 +80,16 @@ __device__ __forceinline__ void store(__nv_bfloat16* to, const Values<VEC>& v) {
   }
 }
 
-__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+// silu whose result leaves as T: for bfloat16 by the hardware's exponential and reciprocal (some units of
+// 2^-22 off, far below the rounding that follows).
+template <typename T>
+__device__ __forceinline__ float silu(float x) {
+  return x / (1.f + expf(-x));
+}
+template <>
+__device__ __forceinline__ float silu<__nv_bfloat16>(float x) {
+  return __fdividef(x, 1.f + __expf(-x));
+}
 
 // A value of the projection, its planes added up.
 template <int VEC>
@@ -115,16 +124,14 @@ __global__ void __launch_bounds__(THREADS) ssm_prepare_kernel(const Prepare p) {
       }
       return;
     }
-    const int h = (x_block - p.z_blocks) * THREADS + threadIdx.x;
-    if (h >= p.heads) return;
-    const float bias = p.dt_bias[h], rate = expf(p.a_log[h]);
-    for (int t = 0; t < tokens; ++t) {
-      const size_t token = (size_t)first + t0 + t;
-      const float x = projected<1>(p, token, p.dt_off + h).x[0] + bias;
-      const float step = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
-      p.step[token * p.heads + h] = step;
-      p.log_decay[token * p.heads + h] = -rate * step;
-    }
+    const int e = (x_block - p.z_blocks) * THREADS + threadIdx.x;       // a head of a token
+    if (e >= tokens * p.heads) return;
+    const int t = e / p.heads, h = e - t * p.heads;
+    const size_t token = (size_t)first + t0 + t;
+    const float x = projected<1>(p, token, p.dt_off + h).x[0] + p.dt_bias[h];
+    const float step = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+    p.step[token * p.heads + h] = step;
+    p.log_decay[token * p.heads + h] = -expf(p.a_log[h]) * step;
     return;
   }
   const int c = (x_block * THREADS + threadIdx.x) * VEC;
@@ -171,7 +178,7 @@ __global__ void __launch_bounds__(THREADS) ssm_prepare_kernel(const Prepare p) {
 #pragma unroll
           for (int v = 0; v < VEC; ++v) acc.x[v] = fmaf(w[j][v], window[j].x[v], acc.x[v]);
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) acc.x[v] = silu(acc.x[v]);
+        for (int v = 0; v < VEC; ++v) acc.x[v] = silu<T>(acc.x[v]);
         store<VEC>(out + (size_t)(t1 + i) * p.channels, acc);
       }
     }
@@ -184,7 +191,7 @@ __global__ void __launch_bounds__(THREADS) ssm_prepare_kernel(const Prepare p) {
         for (int v = 0; v < VEC; ++v) acc.x[v] = fmaf(p.taps_w[(size_t)(c + v) * taps + j], u.x[v], acc.x[v]);
       }
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) acc.x[v] = silu(acc.x[v]);
+      for (int v = 0; v < VEC; ++v) acc.x[v] = silu<T>(acc.x[v]);
       store<VEC>(out + (size_t)t * p.channels, acc);
     }
   }
@@ -241,7 +248,7 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) gated_group_norm_kernel(cons
     if ((lane + k * LANES) * VEC >= p.size) break;
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
-      const float gated = ys[k].x[j] * silu(gs[k].x[j]), v = p.gate_first ? gated : ys[k].x[j];
+      const float gated = ys[k].x[j] * silu<T>(gs[k].x[j]), v = p.gate_first ? gated : ys[k].x[j];
       squares = fmaf(v, v, squares);
       ys[k].x[j] = gated;
     }
@@ -251,7 +258,7 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) gated_group_norm_kernel(cons
     if (p.gate_first) {
       const Values<VEC> g = load<VEC>(gate + i);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) v.x[j] *= silu(g.x[j]);
+      for (int j = 0; j < VEC; ++j) v.x[j] *= silu<T>(g.x[j]);
     }
 #pragma unroll
     for (int j = 0; j < VEC; ++j) squares = fmaf(v.x[j], v.x[j], squares);
@@ -282,7 +289,7 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) gated_group_norm_kernel(cons
     const Values<VEC> g = load<VEC>(gate + i);
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
-      v.x[j] = v.x[j] * silu(g.x[j]) * scale;
+      v.x[j] = v.x[j] * silu<T>(g.x[j]) * scale;
       if (p.weight != nullptr) v.x[j] *= p.weight[c0 + i + j];
     }
     store<VEC>(out + i, v);
@@ -326,7 +333,7 @@ PAE_EXPORT int pae_ssm_prepare(void* u, float* step, float* log_decay, float* z,
   const int vec = wide ? 4 : 1;
   p.u_blocks = (channels + THREADS * vec - 1) / (THREADS * vec);
   p.z_blocks = z != nullptr ? (z_cols + THREADS * vec - 1) / (THREADS * vec) : 0;
-  const dim3 grid(p.u_blocks + p.z_blocks + (heads + THREADS - 1) / THREADS, (max_q_len + TOKENS - 1) / TOKENS, entries);
+  const dim3 grid(p.u_blocks + p.z_blocks + (heads * (max_q_len < TOKENS ? max_q_len : TOKENS) + THREADS - 1) / THREADS, (max_q_len + TOKENS - 1) / TOKENS, entries);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == kF32 && wide) launch_prepare<float, 4>(p, grid, s);
   else if (dtype == kF32) launch_prepare<float, 1>(p, grid, s);
