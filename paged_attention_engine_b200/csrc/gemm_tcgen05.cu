@@ -172,6 +172,7 @@ __device__ __forceinline__ void store_row_chunk(const Params& p, int row, int co
 
 // A gated linear unit in the epilogue: 16 gate columns and the 16 up columns that follow them give 16
 // outputs. Gate and up are rounded to bfloat16 first, as the unfused path stores them.
+template <int GATE>
 __device__ __forceinline__ void store_swiglu_chunk(const Params& p, int row, int col0, const float* g, const float* u) {
   __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)row * p.ld_out + (col0 >> 1);
   uint4 w0, w1;
@@ -182,7 +183,7 @@ __device__ __forceinline__ void store_swiglu_chunk(const Params& p, int row, int
   for (int i = 0; i < 16; ++i) {
     const float gg = __bfloat162float(__float2bfloat16_rn(g[i]));
     const float uu = __bfloat162float(__float2bfloat16_rn(u[i]));
-    r[i] = gated(gg, uu, p.gate_kind);
+    r[i] = gated(gg, uu, GATE);
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -467,7 +468,9 @@ __device__ __forceinline__ void mbar_arrive(uint32_t bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
 }
 
-template <int PBN>
+// GATE: the gate's activation of the gated epilogue, known when compiled (a choice at run time in that
+// epilogue cost the SiLU models 1 % of a step).
+template <int PBN, int GATE>
 __global__ void __launch_bounds__(PERSISTENT_THREADS) gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a,
                                                                           const __grid_constant__ CUtensorMap map_b,
                                                                           const Params p, int tiles_a, int tiles_b) {
@@ -674,7 +677,7 @@ __global__ void __launch_bounds__(PERSISTENT_THREADS) gemm_tcgen05_persistent_ke
           tmem_load16(lane_address + c0, gate);
           tmem_load16(lane_address + c0 + 16, up);
           const int col0 = tile_b * PBN + c0;
-          if (row < rows_end && col0 < p.rows_b) store_swiglu_chunk(p, row, col0, gate, up);
+          if (row < rows_end && col0 < p.rows_b) store_swiglu_chunk<GATE>(p, row, col0, gate, up);
         }
       } else {
 #pragma unroll 1
@@ -728,7 +731,7 @@ int sm_count() {
   return count;
 }
 
-template <int PBN>
+template <int PBN, int GATE>
 int launch_persistent_with(const Params& p, const void* a, const void* b, int k, cudaStream_t stream) {
   using T = PTile<PBN>;
   CUtensorMap map_a, map_b;
@@ -736,14 +739,14 @@ int launch_persistent_with(const Params& p, const void* a, const void* b, int k,
   if (int err = tensor_map(&map_b, b, p.group_tiles != nullptr ? p.rows_b * p.groups : p.rows_b, k, PBN)) return err;
   static bool configured = false;
   if (!configured) {
-    cudaError_t err = cudaFuncSetAttribute(gemm_tcgen05_persistent_kernel<PBN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)T::SMEM_BYTES);
+    cudaError_t err = cudaFuncSetAttribute(gemm_tcgen05_persistent_kernel<PBN, GATE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)T::SMEM_BYTES);
     if (err != cudaSuccess) return fail(100, "linear_tcgen05: %s", cudaGetErrorString(err));
     configured = true;
   }
   const int tiles_a = (p.rows_a + BM - 1) / BM, tiles_b = (p.rows_b + PBN - 1) / PBN;
   const int items = tiles_a * tiles_b * (p.planes > 1 ? p.planes : 1);
   const int blocks = items < sm_count() ? items : sm_count();
-  launch_kernel(gemm_tcgen05_persistent_kernel<PBN>, dim3(blocks), PERSISTENT_THREADS, T::SMEM_BYTES, stream, map_a, map_b, p, tiles_a, tiles_b);
+  launch_kernel(gemm_tcgen05_persistent_kernel<PBN, GATE>, dim3(blocks), PERSISTENT_THREADS, T::SMEM_BYTES, stream, map_a, map_b, p, tiles_a, tiles_b);
   return check_launch("linear_tcgen05");
 }
 
@@ -777,11 +780,17 @@ int persistent_width(const Params& p) {
 
 int launch_persistent(const Params& p, const void* a, const void* b, int k, cudaStream_t stream) {
   const int best = persistent_width(p);
-  if (best == 192) return launch_persistent_with<192>(p, a, b, k, stream);
-  if (best == 176) return launch_persistent_with<176>(p, a, b, k, stream);
-  if (best == 128) return launch_persistent_with<128>(p, a, b, k, stream);
-  if (best == 64) return launch_persistent_with<64>(p, a, b, k, stream);
-  return launch_persistent_with<256>(p, a, b, k, stream);
+  if (p.swiglu && p.gate_kind == kGateRelu) {
+    if (best == 192) return launch_persistent_with<192, kGateRelu>(p, a, b, k, stream);
+    if (best == 128) return launch_persistent_with<128, kGateRelu>(p, a, b, k, stream);
+    if (best == 64) return launch_persistent_with<64, kGateRelu>(p, a, b, k, stream);
+    return launch_persistent_with<256, kGateRelu>(p, a, b, k, stream);
+  }
+  if (best == 192) return launch_persistent_with<192, kGateSilu>(p, a, b, k, stream);
+  if (best == 176) return launch_persistent_with<176, kGateSilu>(p, a, b, k, stream);
+  if (best == 128) return launch_persistent_with<128, kGateSilu>(p, a, b, k, stream);
+  if (best == 64) return launch_persistent_with<64, kGateSilu>(p, a, b, k, stream);
+  return launch_persistent_with<256, kGateSilu>(p, a, b, k, stream);
 }
 
 int check_operands(const void* x, const void* w, int k) {

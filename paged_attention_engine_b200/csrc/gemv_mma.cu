@@ -84,7 +84,10 @@ __device__ __forceinline__ void tma_load_chunks(uint32_t dst, const CUtensorMap*
       : "memory");
 }
 
-enum Kind : int { QKV = 0, RESIDUAL = 1, GATE_UP = 2 };
+// GATE_RELU is gate|up with the rectifier: a kind of its own, because a choice at run time in the
+// epilogue cost a decode step of the SiLU models 1.2 %.
+enum Kind : int { QKV = 0, RESIDUAL = 1, GATE_UP = 2, GATE_RELU = 3 };
+__host__ __device__ constexpr bool is_gate(int kind) { return kind == GATE_UP || kind == GATE_RELU; }
 
 struct Params {
   const __nv_bfloat16* x;        // [tokens, k]
@@ -95,7 +98,6 @@ struct Params {
   // RESIDUAL
   const __nv_bfloat16* residual; // [tokens, n] or null
   __nv_bfloat16* out;            // RESIDUAL: [tokens, n]; GATE_UP: [tokens, n / 2]; QKV: [tokens, n]
-  int gate_kind;                 // GATE_UP: SiLU or the rectifier
   // QKV
   const float* bias;             // [n] or null
   const float* rotary;           // [tokens, d]: cosines then sines, or null
@@ -119,7 +121,7 @@ __device__ __forceinline__ int weight_row(const Params& p, int tile, int r) {
     const int head = tile / per_head, j0 = (tile - head * per_head) * 8;
     return head * p.d + (r < 8 ? j0 : half + j0);
   }
-  if (KIND == GATE_UP) {
+  if (is_gate(KIND)) {
     // rows alternate in blocks of 16 gate, 16 up; tile t holds gate rows 8t..8t+7 of the intermediate size
     const int j = tile * 8;
     return (j >> 4) * 32 + (j & 15) + (r < 8 ? 0 : 16);
@@ -158,7 +160,7 @@ __global__ void __launch_bounds__(WARPS * 32) gemv_kernel(const __grid_constant_
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t4 = lane & 3;
   const int tile = SPLIT ? (int)blockIdx.x : (int)blockIdx.x * WARPS + warp;
-  const int tiles = KIND == QKV ? (p.n / p.d) * (p.d >> 4) : (KIND == GATE_UP ? p.n / 16 : (p.n + ROWS - 1) / ROWS);
+  const int tiles = KIND == QKV ? (p.n / p.d) * (p.d >> 4) : (is_gate(KIND) ? p.n / 16 : (p.n + ROWS - 1) / ROWS);
   const bool live = tile < tiles;
   const int chunks = p.k / CHUNK;
   // this warp's chunks of K
@@ -439,10 +441,10 @@ __global__ void __launch_bounds__(WARPS * 32) gemv_kernel(const __grid_constant_
             to[half + f] = hi16;
           }
         }
-      } else if (KIND == GATE_UP) {
+      } else if (is_gate(KIND)) {
         const int j = tile * 8 + g;
         const float gate = __bfloat162float(__float2bfloat16_rn(lo)), up = __bfloat162float(__float2bfloat16_rn(hi));
-        p.out[(size_t)token * (p.n >> 1) + j] = __float2bfloat16_rn(gated(gate, up, p.gate_kind));
+        p.out[(size_t)token * (p.n >> 1) + j] = __float2bfloat16_rn(gated(gate, up, KIND == GATE_RELU ? kGateRelu : kGateSilu));
       } else {
         const int row_lo = tile * ROWS + g, row_hi = row_lo + 8;
         if (row_lo < p.n) {
@@ -594,7 +596,7 @@ int pick_shape(int k, long blocks, bool* at_once = nullptr) {
   static constexpr int NORMED_ORDER[NUM_SHAPES] = {3, 0, 2, 4, 1}, PLAIN_ORDER[NUM_SHAPES] = {2, 0, 4, 1, 3};
   for (int at = 0; at < NUM_SHAPES; ++at) {
     const int i = NORMED ? NORMED_ORDER[at] : PLAIN_ORDER[at];
-    if (g_forced[KIND] >= 0 && i != g_forced[KIND]) continue;
+    if (g_forced[is_gate(KIND) ? GATE_UP : KIND] >= 0 && i != g_forced[is_gate(KIND) ? GATE_UP : KIND]) continue;
     const size_t bytes = shape_bytes<KIND, NT8, SPLIT, NORMED>(i, k);
     if (bytes > (size_t)SMEM_LIMIT) continue;
     if (fits < 0) fits = i;
@@ -710,8 +712,8 @@ PAE_EXPORT int pae_linear_swiglu_few_tokens(void* out, const void* x, const void
   p.norm_weight = norm_weight;
   p.eps = eps;
   p.out = (__nv_bfloat16*)out;
-  p.gate_kind = gate_kind;
   p.error = error;
+  if (gate_kind == kGateRelu) return launch_tokens<GATE_RELU, false>(p, w, two_inter / 16, (cudaStream_t)stream);
   return launch_tokens<GATE_UP, false>(p, w, two_inter / 16, (cudaStream_t)stream);
 }
 
