@@ -19,6 +19,7 @@ from .model_spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
 from .bidonex import BidonexConfig
 from .finezen import FinezenConfig
 from .getozen import GetozenConfig
+from .luzevik import LuzevikConfig
 from .qwen2 import Qwen2Config
 from .pukerax import PukeraxConfig
 from .zugarax import ZugaraxConfig
@@ -529,3 +530,93 @@ def getozen_spec(cfg: GetozenConfig) -> ModelSpec:
 
 
 register_architecture("Getozen", GetozenConfig, getozen_spec)
+
+
+# --------------------------------------------------------------------------- #
+# Luzevik: a scaled token embedding into a float32 residual stream; no norm in front of a sublayer, one
+# behind it, x <- x + rms(f(x)); the mixer a latent attention (a query latent, a rotated key part whose
+# channels pair half a span apart, a learned sink per head; a layer may read an earlier layer's
+# latent), or a grouped-query attention (biases, q and k normed per head, linearly scaled frequencies)
+# and a gated delta rule side by side, each output normed over the width, half their sum; the
+# feed-forward gated, dense with the tanh form of GELU or a mixture of SiLU experts (a biased router,
+# the softmax over the chosen logits as weights), or absent; RMS norm and the embedding's own table as the head.
+# --------------------------------------------------------------------------- #
+
+# The design has no longest sequence; positions are 32-bit integers.
+LUZEVIK_MAX_POSITIONS = 1 << 30
+# Fixed by the design: the share of either mixer in their sum, and the unit vectors' epsilon.
+LUZEVIK_BRANCH_SCALE = 0.5
+LUZEVIK_KEY_EPS = 1e-6
+
+
+def luzevik_spec(cfg: LuzevikConfig) -> ModelSpec:
+    layers, schedule, unread = [], [], []
+
+    def rotation(rot):
+        scaling = dict(rot.scaling, kind="linear") if rot.scaling is not None else None
+        return {"kind": "scaled_rotary", "dims": rot.dims, "base": rot.base, "scaling": scaling}
+
+    for i, layer in enumerate(cfg.layers):
+        prefix = f"l{i}"
+        m = layer.mixer
+        cache_from = None
+        if layer.type == "latent_attention":
+            mixer = PartSpec(
+                "latent_attention",
+                {
+                    "hidden_size": cfg.width, "num_heads": m.heads, "head_dim": m.dim, "rot_dim": m.rot_dim, "value_dim": m.vdim,
+                    "kv_rank": m.kv_rank, "q_rank": m.q_rank, "scale": m.scale, "norm_eps": cfg.norm_eps, "own_latent": m.kv_from is None,
+                    "pairing": "half", "learned_sink": True, "position_encoding": rotation(m.rot),
+                },
+                f"{prefix}.mix",
+            )
+            cache_from = m.kv_from
+        else:
+            left = {
+                "hidden_size": cfg.width, "num_heads": m.left.heads, "num_kv_heads": m.left.kv_heads, "head_dim": m.left.dim,
+                "value_dim": m.left.vdim, "scale": m.left.scale, "window": 0, "qk_norm_eps": cfg.norm_eps, "qkv_bias": True,
+                "output_gate": False, "pairing": "half", "position_encoding": rotation(m.left.rot),
+            }
+            right = {
+                "hidden_size": cfg.width, "num_heads": m.right.heads, "num_kv_heads": m.right.kv_heads, "head_dim": m.right.dim,
+                "value_dim": m.right.vdim, "conv_taps": m.right.conv, "key_eps": LUZEVIK_KEY_EPS, "norm_eps": cfg.norm_eps,
+            }
+            mixer = PartSpec("side_by_side", {"out_norm_eps": cfg.norm_eps, "hidden_size": cfg.width, "mixers": [
+                {"kind": "gated_window_attention", "params": left, "name": "left", "scale": LUZEVIK_BRANCH_SCALE},
+                {"kind": "gated_delta", "params": right, "name": "right", "scale": LUZEVIK_BRANCH_SCALE}]}, f"{prefix}.mix")
+        norm = lambda name: PartSpec("rms_norm", {"size": cfg.width, "eps": cfg.norm_eps, "out": "engine"}, names={"weight": f"{prefix}.{name}"})
+        parts = dict(mixer=mixer, mixer_out_norm=norm("norm1"))
+        if layer.mlp is not None and layer.mlp.kind == "dense":
+            feed_forward = PartSpec("gated_mlp", {"hidden_size": cfg.width, "intermediate_size": layer.mlp.ff, "activation": "gelu_tanh"},
+                                    f"{prefix}.mlp")
+        elif layer.mlp is not None:
+            feed_forward = PartSpec(
+                "routed_experts",
+                {
+                    "hidden_size": cfg.width, "intermediate_size": layer.mlp.ff, "gated": True, "num_experts": layer.mlp.experts,
+                    "top": layer.mlp.top, "score": "chosen_softmax", "router_bias": True,
+                },
+                f"{prefix}.mlp",
+            )
+        if layer.mlp is not None:
+            parts.update(feed_forward=feed_forward, feed_forward_out_norm=norm("norm2"))
+        else:
+            unread.append(f"{prefix}.norm2")      # the branch that is absent may still have its norm in the checkpoint
+        layers.append(LayerSpec("post_norm_residual" if layer.mlp is not None else "post_norm_residual_mixer", parts))
+        schedule.append(ScheduleEntry(i, cache_from))
+    return ModelSpec(
+        architecture=cfg.architecture,
+        vocab_size=cfg.vocab,
+        hidden_size=cfg.width,
+        max_positions=LUZEVIK_MAX_POSITIONS,
+        embedding=PartSpec("scaled_token_embedding", {"vocab_size": cfg.vocab, "hidden_size": cfg.width, "scale": cfg.embedding_scale},
+                           names={"weight": "embed"}),
+        layers=tuple(layers),
+        schedule=tuple(schedule),
+        final_norm=PartSpec("rms_norm", {"size": cfg.width, "eps": cfg.norm_eps, "out": "engine"}, names={"weight": "final.norm"}),
+        head=PartSpec("lm_head", {"vocab_size": cfg.vocab, "hidden_size": cfg.width, "tied_to": "embed"}),
+        unread=tuple(unread),
+    )
+
+
+register_architecture("Luzevik", LuzevikConfig, luzevik_spec)

@@ -22,7 +22,8 @@
 // results in scratch; `merge` adds them up in their order. Scores and the softmax are float32.
 // Keys are folded in ascending order; a query's result depends on its own keys only. With a
 // window w a query at position i sees the keys i - w < j <= i: a block starts at the tile of its
-// first row's first key, and keys before that key are not fetched (their pages may be gone).
+// first row's first key, and keys before that key are not fetched (their pages may be gone). A sink
+// logit per head (or none) is one more term of the softmax's denominator.
 #include "attention_mma.cuh"
 
 using namespace pae;
@@ -47,6 +48,7 @@ struct LatentParams {
   const int* kv_len;
   int table_width, heads, page_size, D, DV, cols;
   float scale;
+  const float* sink;            // [heads] or null: a logit without key or value in the softmax's denominator
   int splits;
   int window;                   // 0: every earlier key
   float* part_out;              // [requests, heads, splits, DV]
@@ -108,7 +110,11 @@ __global__ void __launch_bounds__(THREADS) latent_kernel(const LatentParams p) {
   float o[MAX_COLS / 8][4];
 #pragma unroll
   for (int n = 0; n < MAX_COLS / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
-  float row_max[2] = {-FLT_MAX, -FLT_MAX}, row_sum[2] = {0.f, 0.f};
+  // a sink is a logit that is always there: the running maximum starts at it, the sum at exp(0); for a
+  // single token, whose rows are heads and whose keys are shared out, the merge adds it once
+  const bool sunk = p.sink != nullptr && !single;
+  const float sink_at = sunk ? p.sink[head0] * LOG2E : -FLT_MAX;
+  float row_max[2] = {sink_at, sink_at}, row_sum[2] = {sunk ? 1.f : 0.f, sunk ? 1.f : 0.f};
   const int row0 = group * GROUP_ROWS;                                 // this group's first row of the block
   const bool working = row0 < rows;                                    // a group without rows only helps to fetch
   const int my_pos[2] = {single ? pos0 : pos0 + row0 + (lane >> 2), single ? pos0 : pos0 + row0 + (lane >> 2) + 8};
@@ -279,7 +285,7 @@ __global__ void latent_merge_kernel(const LatentParams p) {
   const size_t at = ((size_t)b * p.heads + h) * p.splits;
   const int lane = threadIdx.x & 31;
   if (threadIdx.x < 32) {
-    float top = -FLT_MAX;
+    float top = p.sink != nullptr ? p.sink[h] * LOG2E : -FLT_MAX;
     for (int s = lane; s < p.splits; s += 32) top = fmaxf(top, p.part_max[at + s]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
@@ -289,7 +295,7 @@ __global__ void latent_merge_kernel(const LatentParams p) {
     }
     __syncwarp();
     if (lane == 0) {
-      float sum = 0.f;
+      float sum = p.sink != nullptr ? fast_exp2(p.sink[h] * LOG2E - top) : 0.f;
       for (int s = 0; s < p.splits; ++s) sum += p.part_sum[at + s] * weights[s];
       inverse = sum > 0.f ? 1.f / sum : 0.f;
     }
@@ -318,7 +324,7 @@ PAE_EXPORT int pae_attention_latent_mma_supports(int d, int dv) {
 PAE_EXPORT int pae_paged_attention_latent_mma(void* out, const void* q, const void* keys, const int* block_table,
                                               int table_width, const int* q_start, const int* q_pos0, const int* kv_len,
                                               int seqs, int max_q_len, int heads, int d, int dv, int page_size, float scale,
-                                              int window, int splits, float* scratch, void* stream) {
+                                              const float* sink, int window, int splits, float* scratch, void* stream) {
   if (seqs == 0 || max_q_len == 0) return 0;
   if (!pae_attention_latent_mma_supports(d, dv)) return fail(2, "paged_attention_latent_mma: key rows of %d channels with values of %d", d, dv);
   if (splits < 1 || (scratch == nullptr && splits != 1)) return fail(2, "paged_attention_latent_mma: %d splits", splits);
@@ -328,7 +334,7 @@ PAE_EXPORT int pae_paged_attention_latent_mma(void* out, const void* q, const vo
     return fail(2, "paged_attention_latent_mma: an operand does not start on a 16-byte boundary");
   const int cols = (((dv + 3) / 4) + 15) / 16 * 16;
   LatentParams p{(__nv_bfloat16*)out, (const __nv_bfloat16*)q, (const __nv_bfloat16*)keys, block_table, q_start, q_pos0, kv_len,
-                 table_width, heads, page_size, d, dv, cols, scale, splits, window < 0 ? 0 : window, nullptr, nullptr, nullptr};
+                 table_width, heads, page_size, d, dv, cols, scale, sink, splits, window < 0 ? 0 : window, nullptr, nullptr, nullptr};
   if (scratch != nullptr) {
     const size_t units = (size_t)seqs * heads * splits;
     p.part_out = scratch;

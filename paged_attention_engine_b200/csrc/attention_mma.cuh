@@ -92,6 +92,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *(uint32_t*)&v;
 }
 
+// Two float32 numbers as the sum of two bfloat16 pairs: an operand that keeps 16 bits of mantissa.
+__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h2 = __floats2bfloat162_rn(a, b);
+  const float2 back = __bfloat1622float2(h2);
+  hi = *(const uint32_t*)&h2;
+  lo = pack_bf16(a - back.x, b - back.y);
+}
+
 // A tile of rows x D bfloat16 in shared memory; the 16-byte chunk c of row r lives at chunk
 // c ^ swizzle(r), so that the eight rows an ldmatrix reads fall into different banks.
 template <int D>

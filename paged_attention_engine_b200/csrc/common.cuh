@@ -115,10 +115,16 @@ __device__ __forceinline__ int checked_page(int page) {
   return page;
 }
 
-// The gate of a gated linear unit, act(g) * u: SiLU, or the rectifier. The kernels that fold it
+// The gate of a gated linear unit, act(g) * u: SiLU, the rectifier, or the tanh form of GELU. The kernels that fold it
 // into a product's epilogue and the ones that run it alone all call this.
-enum GateKind : int { kGateSilu = 0, kGateRelu = 1 };
+enum GateKind : int { kGateSilu = 0, kGateRelu = 1, kGateGeluTanh = 2 };
+// 0.5 z (1 + tanh w) with w = sqrt(2 / pi) (z + 0.044715 z^3): the half and the tanh are the sigmoid of 2 w.
+__device__ __forceinline__ float gelu_tanh(float z) {
+  const float w = 0.79788456080286535588f * (z + 0.044715f * z * z * z);
+  return z / (1.f + expf(-2.f * w));
+}
 __device__ __forceinline__ float gated(float g, float u, int kind) {
+  if (kind == kGateGeluTanh) return gelu_tanh(g) * u;
   return kind == kGateRelu ? fmaxf(g, 0.f) * u : g / (1.f + expf(-g)) * u;
 }
 

@@ -309,13 +309,6 @@ __device__ __forceinline__ void chunk_decays(const Memory& p, size_t token0, int
   __syncthreads();
 }
 
-__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h2 = __floats2bfloat162_rn(a, b);
-  const float2 back = __bfloat1622float2(h2);
-  hi = *(const uint32_t*)&h2;
-  lo = pack_bf16(a - back.x, b - back.y);
-}
-
 // One chunk's own contribution to the state: an NT x 64 tile of U per block, a warp 32 x 32 of it (NT 64 or 128
 // key channels: the weighted values are split once for all of them).
 constexpr int ST_PITCH = 72;            // bfloat16 elements between rows of a 64-wide tile

@@ -295,7 +295,7 @@ PAE_EXPORT int pae_rotary_qk_cache_write(void* qkv, const float* table, const in
 }
 
 // ------------------------------------------------------------------------------------
-// The middle of a gated feed-forward (engine/model.py:317-320): out[t, i] = act(gate[t, i]) * up[t, i], SiLU or the rectifier,
+// The middle of a gated feed-forward (engine/model.py:317-320): out[t, i] = act(gate[t, i]) * up[t, i], SiLU, the rectifier or the tanh form of GELU,
 // where a row of the input holds the gate in [0, I) and the up projection in [I, 2I).
 // ------------------------------------------------------------------------------------
 template <typename T>

@@ -50,7 +50,7 @@ struct Params {
   int ld_out;        // NORMAL: row pitch of out/residual in elements; SWAPPED: weight rows N
   int out_f32;
   int swiglu;        // NORMAL only: columns come in blocks of 16 gate, 16 up; out[row, n / 2] = act(gate) * up
-  int gate_kind;     // with swiglu: SiLU or the rectifier
+  int gate_kind;     // with swiglu: the gate's activation (GateKind)
   int activation;    // 0: none; 1: exact GELU, 2: tanh GELU, 3: squared ReLU, of the product (+ bias) rounded to the output's type, before the residual
   // q|k|v with rotation and page write in the epilogue (NORMAL, many tokens): out is
   // qkv [tokens, (heads + 2 kv_heads) d]; a tile of 256 columns holds whole heads.
@@ -778,14 +778,18 @@ int persistent_width(const Params& p) {
   return best;
 }
 
+template <int GATE>
+int launch_gated(const Params& p, int width, const void* a, const void* b, int k, cudaStream_t stream) {
+  if (width == 192) return launch_persistent_with<192, GATE>(p, a, b, k, stream);
+  if (width == 128) return launch_persistent_with<128, GATE>(p, a, b, k, stream);
+  if (width == 64) return launch_persistent_with<64, GATE>(p, a, b, k, stream);
+  return launch_persistent_with<256, GATE>(p, a, b, k, stream);
+}
+
 int launch_persistent(const Params& p, const void* a, const void* b, int k, cudaStream_t stream) {
   const int best = persistent_width(p);
-  if (p.swiglu && p.gate_kind == kGateRelu) {
-    if (best == 192) return launch_persistent_with<192, kGateRelu>(p, a, b, k, stream);
-    if (best == 128) return launch_persistent_with<128, kGateRelu>(p, a, b, k, stream);
-    if (best == 64) return launch_persistent_with<64, kGateRelu>(p, a, b, k, stream);
-    return launch_persistent_with<256, kGateRelu>(p, a, b, k, stream);
-  }
+  if (p.swiglu && p.gate_kind == kGateRelu) return launch_gated<kGateRelu>(p, best, a, b, k, stream);
+  if (p.swiglu && p.gate_kind == kGateGeluTanh) return launch_gated<kGateGeluTanh>(p, best, a, b, k, stream);
   if (best == 192) return launch_persistent_with<192, kGateSilu>(p, a, b, k, stream);
   if (best == 176) return launch_persistent_with<176, kGateSilu>(p, a, b, k, stream);
   if (best == 128) return launch_persistent_with<128, kGateSilu>(p, a, b, k, stream);
@@ -803,7 +807,7 @@ int check_operands(const void* x, const void* w, int k) {
 
 // out[tokens, n] = x[tokens, k] . w[n, k]^T (+ bias[n]) (+ residual[tokens, n]); x, w, residual
 // bfloat16, bias float32, out bfloat16 or float32 (then residual is float32 too).
-// out[tokens, n / 2] = act(gate) * up (gate_kind 0: SiLU, 1: the rectifier) where x . w^T gives gate and up in alternating blocks of 16
+// out[tokens, n / 2] = act(gate) * up (gate_kind 0: SiLU, 1: the rectifier, 2: the tanh form of GELU) where x . w^T gives gate and up in alternating blocks of 16
 // columns (w's rows are laid out that way); many tokens only (the persistent kernel). n is a
 // multiple of 32 and at least 256.
 PAE_EXPORT int pae_linear_swiglu_tcgen05(void* out, const void* x, const void* w, int tokens, int n, int k, int gate_kind,

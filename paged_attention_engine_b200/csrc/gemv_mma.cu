@@ -16,7 +16,7 @@
 //             the token (the product runs over x * norm weight; rsqrt(mean x^2 + eps) is one
 //             factor per token and is applied to the sums), bias, rounding, rotation, page write.
 //   gate|up   8 gate rows and their 8 up rows (the weight's rows alternate in blocks of 16):
-//             epilogue = scale, rounding, act(gate) * up (SiLU or the rectifier).
+//             epilogue = scale, rounding, act(gate) * up (SiLU, the rectifier or the tanh form of GELU).
 //   o, down   16 neighbouring rows; epilogue = + residual, rounding.
 //
 // Weights: every warp runs a ring of its own, filled by TMA and watched through one mbarrier
@@ -84,10 +84,11 @@ __device__ __forceinline__ void tma_load_chunks(uint32_t dst, const CUtensorMap*
       : "memory");
 }
 
-// GATE_RELU is gate|up with the rectifier: a kind of its own, because a choice at run time in the
-// epilogue cost a decode step of the SiLU models 1.2 %.
-enum Kind : int { QKV = 0, RESIDUAL = 1, GATE_UP = 2, GATE_RELU = 3 };
-__host__ __device__ constexpr bool is_gate(int kind) { return kind == GATE_UP || kind == GATE_RELU; }
+// GATE_RELU and GATE_GELU are gate|up with the rectifier and with the tanh form of GELU: kinds of their own,
+// because a choice at run time in the epilogue cost a decode step of the SiLU models 1.2 %.
+enum Kind : int { QKV = 0, RESIDUAL = 1, GATE_UP = 2, GATE_RELU = 3, GATE_GELU = 4 };
+__host__ __device__ constexpr bool is_gate(int kind) { return kind >= GATE_UP; }
+__host__ __device__ constexpr int gate_of(int kind) { return kind == GATE_RELU ? kGateRelu : kind == GATE_GELU ? kGateGeluTanh : kGateSilu; }
 
 struct Params {
   const __nv_bfloat16* x;        // [tokens, k]
@@ -444,7 +445,7 @@ __global__ void __launch_bounds__(WARPS * 32) gemv_kernel(const __grid_constant_
       } else if (is_gate(KIND)) {
         const int j = tile * 8 + g;
         const float gate = __bfloat162float(__float2bfloat16_rn(lo)), up = __bfloat162float(__float2bfloat16_rn(hi));
-        p.out[(size_t)token * (p.n >> 1) + j] = __float2bfloat16_rn(gated(gate, up, KIND == GATE_RELU ? kGateRelu : kGateSilu));
+        p.out[(size_t)token * (p.n >> 1) + j] = __float2bfloat16_rn(gated(gate, up, gate_of(KIND)));
       } else {
         const int row_lo = tile * ROWS + g, row_hi = row_lo + 8;
         if (row_lo < p.n) {
@@ -698,7 +699,7 @@ PAE_EXPORT int pae_linear_few_tokens(void* out, const void* x, const void* w, co
   return launch_tokens<RESIDUAL, true>(p, w, (n + ROWS - 1) / ROWS, (cudaStream_t)stream);
 }
 
-// out[token, inter] = act(g) * u (gate_kind 0: SiLU, 1: the rectifier) with g, u = RMSNorm(x) . (gate, up rows of w)^T, each rounded to
+// out[token, inter] = act(g) * u (gate_kind 0: SiLU, 1: the rectifier, 2: the tanh form of GELU) with g, u = RMSNorm(x) . (gate, up rows of w)^T, each rounded to
 // bfloat16 first; w [2 inter, k] with rows alternating in blocks of 16 gate, 16 up.
 PAE_EXPORT int pae_linear_swiglu_few_tokens(void* out, const void* x, const void* w, const float* norm_weight, float eps,
                                             int tokens, int two_inter, int k, int gate_kind, int* error, void* stream) {
@@ -714,6 +715,7 @@ PAE_EXPORT int pae_linear_swiglu_few_tokens(void* out, const void* x, const void
   p.out = (__nv_bfloat16*)out;
   p.error = error;
   if (gate_kind == kGateRelu) return launch_tokens<GATE_RELU, false>(p, w, two_inter / 16, (cudaStream_t)stream);
+  if (gate_kind == kGateGeluTanh) return launch_tokens<GATE_GELU, false>(p, w, two_inter / 16, (cudaStream_t)stream);
   return launch_tokens<GATE_UP, false>(p, w, two_inter / 16, (cudaStream_t)stream);
 }
 

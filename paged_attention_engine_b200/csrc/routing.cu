@@ -7,6 +7,8 @@
 //            the lower index first among equals
 //   weights  w_e = s_e / (sum of the chosen s + eps) * scale for the chosen, 0 for the others;
 //            or, not normalized, w_e = s_e * scale
+//   or        (chosen softmax) s = z itself, the same choice, w = softmax over the chosen z alone * scale
+// z may include a bias per expert, which is added to the router's sums.
 //
 // One warp per token; all arithmetic float32. The kernel leaves the chosen experts, their weights
 // and, when asked, the dense row of weights [total experts].
@@ -21,13 +23,16 @@ namespace {
 constexpr int WARPS = 4;
 constexpr int MAX_PER_LANE = 16;      // 512 experts
 
+enum Score : int { SOFTMAX = 0, SIGMOID = 1, CHOSEN_SOFTMAX = 2 };
+
 struct Route {
   const float* logits;       // [splits, tokens, ld], of which the first `total` columns: the planes of a split product are added in their order
+  const float* bias;         // [total] or null: part of the logits
   const float* correction;   // [total] or null
   int* chosen;               // [tokens, top]
   float* weights;            // [tokens, top]
   float* dense;              // [tokens, total] or null
-  int tokens, total, top, groups, keep, sigmoid;
+  int tokens, total, top, groups, keep, score;
   float eps, scale;
   int splits, ld, normalize;
 };
@@ -61,11 +66,13 @@ __global__ void __launch_bounds__(WARPS * 32) route_kernel(const Route p) {
     if (e < p.total) {
       float sum = z[e];
       for (int k = 1; k < p.splits; ++k) sum += z[(size_t)k * p.tokens * p.ld + e];
-      s[j] = sum;
+      s[j] = p.bias != nullptr ? sum + p.bias[e] : sum;
     }
     top = fmaxf(top, s[j]);
   }
-  if (p.sigmoid) {
+  if (p.score == CHOSEN_SOFTMAX) {
+    // the logits as they are
+  } else if (p.score == SIGMOID) {
 #pragma unroll
     for (int j = 0; j < PER_LANE; ++j) s[j] = lane + 32 * j < p.total ? 1.f / (1.f + expf(-s[j])) : 0.f;
   } else {
@@ -113,7 +120,7 @@ __global__ void __launch_bounds__(WARPS * 32) route_kernel(const Route p) {
       if (group_score[e / size] != FLT_MAX) choice[e] = -INFINITY;
     __syncwarp();
   }
-  float chosen_sum = 0.f;
+  float chosen_sum = 0.f, first_score = 0.f;
   int mine = 0;                                         // bit j: this lane's expert lane + 32 j is chosen
   for (int k = 0; k < p.top; ++k) {
     float v = -INFINITY;
@@ -132,6 +139,10 @@ __global__ void __launch_bounds__(WARPS * 32) route_kernel(const Route p) {
         if (j == (i >> 5)) score = s[j];
     }
     score = __shfl_sync(0xffffffffu, score, i == INT_MAX ? 0 : (i & 31));
+    if (p.score == CHOSEN_SOFTMAX) {
+      if (k == 0) first_score = score;                  // without a correction the largest; any chosen one serves as the reference
+      score = expf(score - first_score);
+    }
     chosen_sum += score;                                // in the order of the choice, the same on every lane
     if (lane == 0) {
       p.chosen[(size_t)t * p.top + k] = i == INT_MAX ? 0 : i;
@@ -388,8 +399,8 @@ __global__ void expert_combine4_kernel(float* __restrict__ out, const float* __r
 
 }  // namespace
 
-PAE_EXPORT int pae_route(int* chosen, float* weights, float* dense, const float* logits, int splits, int ld, const float* correction, int tokens,
-                         int total, int top, int groups, int keep, int sigmoid, int normalize, float eps, float scale, void* stream) {
+PAE_EXPORT int pae_route(int* chosen, float* weights, float* dense, const float* logits, int splits, int ld, const float* bias, const float* correction, int tokens,
+                         int total, int top, int groups, int keep, int score, int normalize, float eps, float scale, void* stream) {
   if (tokens == 0) return 0;
   if (total < 1 || total > 32 * MAX_PER_LANE) return fail(2, "route: %d experts (1 to %d)", total, 32 * MAX_PER_LANE);
   if (top < 1 || top > total) return fail(2, "route: %d of %d experts", top, total);
@@ -397,7 +408,8 @@ PAE_EXPORT int pae_route(int* chosen, float* weights, float* dense, const float*
     return fail(2, "route: %d experts in %d groups of which %d are kept, %d chosen", total, groups, keep, top);
   if (splits < 1) return fail(2, "route: %d planes of logits", splits);
   if (ld < total) return fail(2, "route: %d experts in rows of %d", total, ld);
-  Route p{logits, correction, chosen, weights, dense, tokens, total, top, groups, keep, sigmoid, eps, scale, splits, ld, normalize};
+  if (score < SOFTMAX || score > CHOSEN_SOFTMAX) return fail(2, "route: score kind %d", score);
+  Route p{logits, bias, correction, chosen, weights, dense, tokens, total, top, groups, keep, score, eps, scale, splits, ld, normalize};
   const size_t smem = sizeof(float) * WARPS * (size_t)(total + groups);
   const unsigned blocks = (tokens + WARPS - 1) / WARPS;
   cudaStream_t s = (cudaStream_t)stream;

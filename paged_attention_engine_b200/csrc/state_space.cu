@@ -5,6 +5,7 @@
 // product, added here in their order), per token:
 //   u_c = silu(bias_c + sum_j taps[c, j] raw[t - taps + 1 + j, c])      every channel of x, B and C
 //   step_h = softplus(dt_h + dt_bias_h)          log_decay_h = -exp(A_log_h) step_h
+//   beta_h = sigmoid(b_h)                        for a mixer that has such columns (the gated delta rule)
 // The last taps - 1 raw rows of a request are kept as per-request state, so a portion's first tokens
 // read the rows before it; zeros stand before a sequence's start. The thread that owns a channel of
 // a portion's first tokens reads the old rows, uses them, and puts the portion's last rows in
@@ -34,12 +35,13 @@ struct Prepare {
   void* u;                  // [tokens, channels]
   float* step;              // [tokens, heads]
   float* log_decay;         // [tokens, heads]
+  float* beta;              // [tokens, heads] or null
   float* z;                 // [tokens, z_cols]: the gate's columns, summed; null: they stay in proj
   const int* q_start;
   const int* q_pos0;
   const int* state_slot;
   long long slot_stride, plane;
-  int planes, ld, z_off, z_cols, u_off, channels, dt_off, heads, taps;
+  int planes, ld, z_off, z_cols, u_off, channels, dt_off, beta_off, heads, taps;
   int u_blocks, z_blocks;   // blockIdx.x: channels of u, then of z, then heads of the block's tokens
 };
 
@@ -132,6 +134,7 @@ __global__ void __launch_bounds__(THREADS) ssm_prepare_kernel(const Prepare p) {
     const float step = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
     p.step[token * p.heads + h] = step;
     p.log_decay[token * p.heads + h] = -expf(p.a_log[h]) * step;
+    if (p.beta != nullptr) p.beta[token * p.heads + h] = 1.f / (1.f + expf(-projected<1>(p, token, p.beta_off + h).x[0]));
     return;
   }
   const int c = (x_block * THREADS + threadIdx.x) * VEC;
@@ -309,9 +312,9 @@ bool aligned16(const void* ptr) { return (((uintptr_t)ptr) & 15) == 0; }
 }  // namespace
 
 // proj float32 [planes][tokens, ld] with z (z_cols columns), u (channels) and dt (heads) at the given
-// offsets; u [tokens, channels] in `dtype`; step and log_decay float32 [tokens, heads]; z float32 [tokens,
+// offsets; u [tokens, channels] in `dtype`; step and log_decay float32 [tokens, heads]; beta likewise or null; z float32 [tokens,
 // z_cols] or null. state: slot s holds [taps - 1, channels] floats at state + s * slot_stride.
-PAE_EXPORT int pae_ssm_prepare(void* u, float* step, float* log_decay, float* z, float* state, long long slot_stride, const float* proj,
+PAE_EXPORT int pae_ssm_prepare(void* u, float* step, float* log_decay, float* beta, int beta_off, float* z, float* state, long long slot_stride, const float* proj,
                                int planes, int ld, int z_off, int z_cols, int u_off, int channels, int dt_off, int heads,
                                const float* taps_w, int taps, const float* bias, const float* dt_bias, const float* a_log,
                                const int* q_start, const int* q_pos0, const int* state_slot, int tokens, int entries, int max_q_len,
@@ -323,7 +326,7 @@ PAE_EXPORT int pae_ssm_prepare(void* u, float* step, float* log_decay, float* z,
     return fail(3, "ssm_prepare: %d requests of up to %d tokens exceed one launch", entries, max_q_len);
   Prepare p{};
   p.proj = proj, p.taps_w = taps_w, p.bias = bias, p.dt_bias = dt_bias, p.a_log = a_log;
-  p.state = state, p.u = u, p.step = step, p.log_decay = log_decay, p.z = z;
+  p.state = state, p.u = u, p.step = step, p.log_decay = log_decay, p.z = z, p.beta = beta, p.beta_off = beta_off;
   p.q_start = q_start, p.q_pos0 = q_pos0, p.state_slot = state_slot;
   p.slot_stride = slot_stride, p.plane = (long long)tokens * ld;
   p.planes = planes, p.ld = ld, p.z_off = z_off, p.z_cols = z_cols, p.u_off = u_off, p.channels = channels;

@@ -58,6 +58,8 @@ FAMILIES: dict[str, list[str]] = {
     "routing": ["routing.cu", "common.cuh"],
     "dyt": ["dyt.cu", "common.cuh"],
     "decay_memory": ["decay_memory.cu", "attention_mma.cuh", "common.cuh"],
+    "gated_delta": ["gated_delta.cu", "attention_mma.cuh", "common.cuh"],
+    "post_norm": ["post_norm.cu", "common.cuh"],
     "state_space": ["state_space.cu", "common.cuh"],
     "attention_decode_noalloc": [
         "attention_decode_noalloc.cu", "attention_decode_noalloc.h", "attention_mma.cuh", "common.cuh",

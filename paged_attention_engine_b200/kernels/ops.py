@@ -247,8 +247,51 @@ class PendingResidual:
         return self.x.device
 
 
+class PendingBranches:
+    """A sublayer's output that is a sum of branches side by side, each normed over the width first: sum_b
+    scale_b * rms(y_b) * w_b, float32, not yet made. `branches` holds (y, weight, scale), every y a tensor
+    or a product that is still in its splits."""
+
+    def __init__(self, branches, eps: float) -> None:
+        self.branches, self.eps = list(branches), float(eps)
+        self.dtype = torch.float32
+        self.value = None
+
+    @property
+    def shape(self):
+        return self.branches[0][0].shape
+
+    @property
+    def device(self):
+        return self.branches[0][0].device
+
+
+class PendingPostNorm:
+    """A float32 residual stream x + mult * rms(y) * weight whose sum has not been made: `post_norm_add`
+    returns one, and the read that follows (`stream_read`, or the last norm) makes the sum inside its own
+    kernel; anything else calls `materialized`, which runs the sum alone. y is a sublayer's output: a
+    tensor, a product that is still in its splits, or PendingBranches."""
+
+    def __init__(self, x, y, weight, eps: float, mult: float) -> None:
+        self.x, self.y, self.weight, self.eps, self.mult = x, y, weight, float(eps), float(mult)
+        self.dtype = torch.float32
+        self.value = None
+
+    @property
+    def shape(self):
+        return self.x.shape
+
+    @property
+    def device(self):
+        return self.x.device
+
+
 def materialized(x):
-    """The tensor that `x` stands for (x itself unless it is a PendingSum, a PendingNorm, PendingStreams or a PendingResidual)."""
+    """The tensor that `x` stands for (x itself unless it is one of the Pending classes above)."""
+    if isinstance(x, (PendingPostNorm, PendingBranches)):
+        if x.value is None:
+            _post_norm_step(x)
+        return x.value
     if isinstance(x, PendingResidual):
         if x.value is None:
             _dyt_step(x, None, None)
@@ -802,11 +845,11 @@ def paged_attention(qkv, keys, values, block_table, q_start, q_pos0, kv_len, num
 
 
 # The activations of a gated linear unit's gate.
-GATE_KINDS = {"silu": 0, "relu": 1}
+GATE_KINDS = {"silu": 0, "relu": 1, "gelu_tanh": 2}
 
 
 def silu_mul(gate_up, block: int = 0, gate: str = "silu") -> torch.Tensor:
-    """act(gate) * up (`gate`: "silu" or "relu") of a [tokens, 2 I] product. block 0: gate is columns [0, I) and up [I, 2 I);
+    """act(gate) * up (`gate`: "silu", "relu" or "gelu_tanh") of a [tokens, 2 I] product. block 0: gate is columns [0, I) and up [I, 2 I);
     block b: b gate columns, then their b up columns, and so on (`linear_swiglu`'s weight layout)."""
     tokens, two_i = gate_up.shape
     if two_i % 2 or (block and two_i % (2 * block)):
@@ -843,7 +886,7 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor | N
 
 
 def linear_swiglu(x, weight, gate: str = "silu") -> torch.Tensor:
-    """act(x . Wg^T) (`gate`: "silu" or "relu") * (x . Wu^T) -> [M, I] for a weight from `interleave_gate_up`. With many
+    """act(x . Wg^T) (`gate`: "silu", "relu" or "gelu_tanh") * (x . Wu^T) -> [M, I] for a weight from `interleave_gate_up`. With many
     tokens the activation runs in the product's epilogue; with few, in the kernel that sums the
     splits; otherwise as a kernel of its own. Gate and up are rounded to the engine dtype first in
     every one of them, so all give the same bits."""
@@ -942,6 +985,8 @@ def rms_norm_cast(x, weight: torch.Tensor, eps: float, out_dtype=None) -> torch.
     """x / sqrt(mean(x^2) + eps) * weight over the last axis; x float32 or the engine's dtype, the
     result in `out_dtype` (x's when None)."""
     _need(weight, "rms_norm_cast: weight", torch.float32)
+    if isinstance(x, PendingPostNorm) and x.value is None:
+        return _post_norm_step(x, out_dtype or torch.float32, weight, eps)     # the residual sum and this norm of it as one kernel
     if (isinstance(x, PendingSum) and x.value is None and not x.activation and x.dtype == torch.float32 and fuse_split_sums
             and weight.numel() == x.shape[-1]):
         # the sum of a split product (+ bias + residual) and the norm of the result as one kernel
@@ -1253,7 +1298,7 @@ def paged_attention_scored(q, keys, values, block_table, q_start, q_pos0, kv_len
     out = torch.empty((tokens, num_heads * value_dim), dtype=q.dtype, device=q.device)
     in_keys = values.data_ptr() == keys.data_ptr()        # a key row's leading channels are its value
     if (in_keys and q.dtype == torch.bfloat16 and use_tensor_cores and form != "simt" and num_kv_heads == 1 and not keep_first
-            and not softcap and temp is None and r1 is None and sink is None):
+            and not softcap and temp is None and r1 is None):
         # Many heads over one latent key/value head, causal or windowed (csrc/attention_latent_mma.cu). A request that brings one
         # token is blocks of up to 32 heads; its keys are shared out (two tiles of 64 a block at least) until the launch fills the GPU once.
         lib = _lib("attention_latent_mma")
@@ -1268,7 +1313,7 @@ def paged_attention_scored(q, keys, values, block_table, q_start, q_pos0, kv_len
                 scratch = torch.empty(seqs * num_heads * splits * (value_dim + 2), dtype=torch.float32, device=q.device)
             _check(lib, lib.pae_paged_attention_latent_mma(
                 _ptr(out), _ptr(q), _ptr(keys), _ptr(block_table), block_table.shape[1], _ptr(q_start), _ptr(q_pos0), _ptr(kv_len),
-                seqs, max_q_len, num_heads, head_dim, value_dim, page_size, scale, int(window or 0), splits, _ptr(scratch), _stream()),
+                seqs, max_q_len, num_heads, head_dim, value_dim, page_size, scale, _ptr(sink), int(window or 0), splits, _ptr(scratch), _stream()),
                 2 if scratch is not None else 1)
             return out
     if (q.dtype == torch.bfloat16 and use_tensor_cores and head_dim in (32, 64, 128) and value_dim in (32, 64, 128)
@@ -1462,6 +1507,85 @@ def join_stream(x, extra):
 
 
 # ----------------------------------------------------------------------------------- #
+# Norms behind a sublayer (csrc/post_norm.cu)
+
+POST_NORM_BRANCHES = 4
+
+
+def _post_norm_step(x, read_dtype=None, read_weight=None, read_eps: float = 0.0):
+    """Runs what is pending in `x` (PendingPostNorm: the branches' norms and sum, the norm behind the
+    sublayer, the residual sum; PendingBranches: their norms and sum; a tensor: nothing) and keeps it in
+    `x.value`; with `read_dtype`, the same kernel leaves the result in that dtype (normed with
+    `read_weight` when given), which is returned."""
+    stream = post = None
+    y, post_eps, mult = x, 0.0, 1.0
+    if isinstance(x, PendingPostNorm):
+        stream, y, post, post_eps, mult = materialized(x.x), x.y, x.weight, x.eps, x.mult
+        _need(stream, "post_norm: the stream", torch.float32)
+    branches, branch_eps = [], 0.0
+    if isinstance(y, PendingBranches) and y.value is None:
+        branches, branch_eps = y.branches, y.eps
+    elif y is not None and (stream is not None or isinstance(y, PendingSum)):
+        branches = [(y, None, 1.0)]
+    else:
+        stream = materialized(y)
+        _need(stream, "post_norm: the stream", torch.float32)
+    if len(branches) > POST_NORM_BRANCHES:
+        raise KernelError(f"post_norm: {len(branches)} branches (up to {POST_NORM_BRANCHES})")
+    outputs, planes, weights, scales = [], [], [], []
+    for out, weight, scale in branches:
+        out, count = _sublayer_output(out)
+        outputs.append(out)
+        planes.append(count)
+        weights.append(weight)
+        scales.append(float(scale))
+    tokens, width = (stream if stream is not None else outputs[0]).shape[-2:]
+    for out in outputs:
+        if tuple(out.shape[-2:]) != (tokens, width):
+            raise KernelError(f"post_norm: a sublayer's output {tuple(out.shape)} for a stream [{tokens}, {width}]")
+    for name, weight in [("a branch", w) for w in weights] + [("the norm behind the sublayer", post), ("the read", read_weight)]:
+        if weight is not None:
+            _need(weight, f"post_norm: weight of {name}", torch.float32)
+            if weight.numel() != width:
+                raise KernelError(f"post_norm: {name} has {weight.numel()} weights for rows of {width}")
+    device = (stream if stream is not None else outputs[0]).device
+    value = torch.empty((tokens, width), dtype=torch.float32, device=device) if branches else stream
+    read = torch.empty((tokens, width), dtype=read_dtype, device=device) if read_dtype is not None else None
+    pad = POST_NORM_BRANCHES - len(outputs)
+    lib = _lib("post_norm")
+    _check(lib, lib.pae_post_norm(
+        _ptr(value if branches else None), _ptr(read), _ptr(stream), len(outputs), *[_ptr(t) for t in outputs], *[None] * pad, *planes,
+        *[1] * pad, *[_ptr(t) for t in weights], *[None] * pad, *scales, *[1.0] * pad, branch_eps, _ptr(post), post_eps, mult,
+        _ptr(read_weight), float(read_eps), tokens, width, _DTYPE_CODE[read_dtype] if read_dtype is not None else 0, _stream()))
+    if isinstance(x, (PendingPostNorm, PendingBranches)):
+        x.value = value
+    return read
+
+
+def normed_branches(branches, eps: float) -> PendingBranches:
+    """sum_b scale_b * rms(y_b) * weight_b for branches (y, weight, scale), float32 [tokens, width], pending:
+    `post_norm_add` takes it along in its own kernel."""
+    return PendingBranches(branches, eps)
+
+
+def post_norm_add(x, y, weight, eps: float, mult: float = 1.0) -> PendingPostNorm:
+    """The stream x + mult * rms(y) * weight, float32, pending: the next `stream_read` or `rms_norm_cast`
+    makes the sum in its own kernel."""
+    return PendingPostNorm(x, y, weight, eps, mult)
+
+
+def stream_read(x, out_dtype) -> torch.Tensor:
+    """A float32 stream in `out_dtype`, what a sublayer without a norm in front reads; a pending residual
+    sum is made on the way (`materialized(x)` then has it)."""
+    if isinstance(x, PendingPostNorm) and x.value is None:
+        if out_dtype == torch.float32:
+            return materialized(x)
+        return _post_norm_step(x, out_dtype)
+    x = materialized(x)
+    return x if x.dtype == out_dtype else _post_norm_step(x, out_dtype)
+
+
+# ----------------------------------------------------------------------------------- #
 # A memory that decays (csrc/decay_memory.cu) and what stands around it (csrc/state_space.cu)
 
 def _state_rows(state, floats: int, what: str):
@@ -1533,17 +1657,74 @@ def decay_memory(q, k, v, state, q_start, state_slot, num_seqs: int, num_heads: 
     return o
 
 
+def gated_delta(q, k, v, log_decay, beta, state, q_start, state_slot, num_seqs: int, num_heads: int, groups: int, key_dim: int,
+                value_dim: int, key_eps: float, q_scale: float = 1.0, max_q_len: int = 1, num_single: int | None = None, multi_index=None,
+                form: str | None = None) -> torch.Tensor:
+    """S <- exp(log_decay) S, u = beta (v - S^T k'), S <- S + k' u^T, o = S^T q' over the step's tokens, k' and q'
+    unit vectors per head (q' times q_scale), from and into the per-request state (float32, [heads,
+    key_dim, value_dim] a slot): see csrc/gated_delta.cu. q, k and v are (tensor [tokens, ld], first
+    column): `groups` query and key heads, `num_heads` value heads; log_decay and beta float32 [tokens,
+    heads]. Single tokens take the step kernel, portions the chunked tensor-core kernels (bfloat16,
+    rows of 16-byte pieces, up to 256 key channels), everything else, and everything when `form` is
+    "scan", goes token after token. -> float32 [tokens, heads * value_dim]."""
+    tokens = q[0].shape[0]
+    rows = []
+    for name, (t, off), width in (("q", q, groups * key_dim), ("k", k, groups * key_dim), ("v", v, num_heads * value_dim)):
+        _need(t, f"gated_delta: {name}", q[0].dtype)
+        if t.dim() != 2 or t.shape[0] != tokens or off < 0 or off + width > t.shape[1]:
+            raise KernelError(f"gated_delta: {name} columns {off}..{off + width} of {tuple(t.shape)} for {tokens} tokens")
+        rows += [t.data_ptr() + off * t.element_size(), int(t.shape[1])]
+    for name, t in (("log_decay", log_decay), ("beta", beta)):
+        _need(t, f"gated_delta: {name}", torch.float32)
+        if t.numel() != tokens * num_heads:
+            raise KernelError(f"gated_delta: {name} has {t.numel()} numbers for {tokens} tokens of {num_heads} heads")
+    _need(q_start, "gated_delta: q_start", torch.int32)
+    _need(state_slot, "gated_delta: state_slot", torch.int32)
+    address, stride = _state_rows(state, num_heads * key_dim * value_dim, "gated_delta")
+    o = torch.empty((tokens, num_heads * value_dim), dtype=torch.float32, device=q[0].device)
+    lib = _lib("gated_delta")
+    what = (_ptr(o), address, stride, *rows, _ptr(log_decay), _ptr(beta), float(key_eps), float(q_scale), _ptr(q_start), _ptr(state_slot))
+    sizes = (num_heads, groups, key_dim, value_dim)
+    code = _code(q[0])
+    singles = num_single if num_single is not None else (num_seqs if max_q_len == 1 else -1)
+    stepped = form != "scan" and address % 16 == 0 and lib.pae_gated_delta_step_supports(key_dim, value_dim, stride) == 1
+    if stepped and singles != 0:
+        _check(lib, lib.pae_gated_delta_step(*what, num_seqs, *sizes, code, _stream()))
+    if singles == num_seqs and stepped:
+        return o
+    chunked = (form != "scan" and use_tensor_cores and code == 1 and address % 16 == 0 and all(r % 16 == 0 for r in rows[::2])
+               and lib.pae_gated_delta_chunked_supports(key_dim, value_dim, rows[1], rows[3], rows[5], stride) == 1)
+    if not chunked or not stepped:
+        _check(lib, lib.pae_gated_delta_scan(*what, num_seqs, *sizes, 1 if stepped else 0, code, _stream()))
+        return o
+    listed = num_seqs
+    if multi_index is not None:
+        _need(multi_index, "gated_delta: multi_index", torch.int32)
+        listed = multi_index.numel()
+    chunk = lib.pae_gated_delta_chunk()
+    units = (tokens // chunk + listed) * num_heads
+    w = torch.empty(units * 2 * chunk * key_dim, dtype=torch.bfloat16, device=o.device)
+    u0 = torch.empty(units * chunk * value_dim, dtype=torch.float32, device=o.device)
+    u = torch.empty(units * 2 * chunk * value_dim, dtype=torch.bfloat16, device=o.device)
+    before = torch.empty(units * 2 * key_dim * value_dim, dtype=torch.bfloat16, device=o.device)
+    vec = torch.empty(units * 2 * chunk, dtype=torch.float32, device=o.device)
+    _check(lib, lib.pae_gated_delta_chunked(*what, _ptr(multi_index), listed, max_q_len, *sizes, _ptr(w), _ptr(u0), _ptr(u), _ptr(before),
+                                            _ptr(vec), _stream()), 3)
+    return o
+
+
 def ssm_prepare(proj, z_off: int, z_cols: int, u_off: int, channels: int, dt_off: int, heads: int, taps_weight, bias, dt_bias, a_log,
-                state, q_start, q_pos0, state_slot, num_seqs: int, max_q_len: int, out_dtype):
+                state, q_start, q_pos0, state_slot, num_seqs: int, max_q_len: int, out_dtype, beta_off: int | None = None):
     """From the fused input projection (float32 [tokens, ld], or the planes of a split product) of a
     selective state space to its recurrence's operands (csrc/state_space.cu): -> (u = silu(causal
     convolution of the `channels` columns at u_off) [tokens, channels] in `out_dtype`, step =
     softplus(dt + dt_bias) and log_decay = -exp(a_log) step, float32 [tokens, heads], and the gate as
-    (rows, first column): the projection itself, or its summed columns). `state` float32 [slots, (taps - 1) *
+    (rows, first column): the projection itself, or its summed columns). With `beta_off`, a fifth: sigmoid of
+    the `heads` columns there, float32 [tokens, heads]. `state` float32 [slots, (taps - 1) *
     channels] is brought up to date."""
     proj, planes = _sublayer_output(proj)
     tokens, ld = int(proj.shape[-2]), int(proj.shape[-1])
-    for off, width in ((z_off, z_cols), (u_off, channels), (dt_off, heads)):
+    for off, width in ((z_off, z_cols), (u_off, channels), (dt_off, heads), (beta_off or 0, heads)):
         if off < 0 or off + width > ld:
             raise KernelError(f"ssm_prepare: columns {off}..{off + width} of rows of {ld}")
     _need(taps_weight, "ssm_prepare: taps", torch.float32)
@@ -1563,13 +1744,15 @@ def ssm_prepare(proj, z_off: int, z_cols: int, u_off: int, channels: int, dt_off
     u = torch.empty((tokens, channels), dtype=out_dtype, device=proj.device)
     step = torch.empty((tokens, heads), dtype=torch.float32, device=proj.device)
     log_decay = torch.empty((tokens, heads), dtype=torch.float32, device=proj.device)
+    beta = torch.empty_like(step) if beta_off is not None else None
     z = torch.empty((tokens, z_cols), dtype=torch.float32, device=proj.device) if planes > 1 else None
     lib = _lib("state_space")
-    _check(lib, lib.pae_ssm_prepare(_ptr(u), _ptr(step), _ptr(log_decay), _ptr(z), address, stride, _ptr(proj), planes, ld, z_off, z_cols,
+    _check(lib, lib.pae_ssm_prepare(_ptr(u), _ptr(step), _ptr(log_decay), _ptr(beta), beta_off or 0, _ptr(z), address, stride, _ptr(proj), planes, ld, z_off, z_cols,
                                     u_off, channels, dt_off, heads, _ptr(taps_weight), taps, _ptr(bias), _ptr(dt_bias), _ptr(a_log),
                                     _ptr(q_start), _ptr(q_pos0), _ptr(state_slot), tokens, num_seqs, max_q_len,
                                     _DTYPE_CODE[out_dtype], _stream()))
-    return u, step, log_decay, (z, 0) if z is not None else (proj.view(tokens, ld), z_off)
+    gate = (z, 0) if z is not None else (proj.view(tokens, ld), z_off)
+    return (u, step, log_decay, gate) if beta is None else (u, step, log_decay, gate, beta)
 
 
 def gated_group_norm(y, gate, gate_off: int, groups: int, eps: float, out_dtype, weight=None, gate_first: bool = False, mult: float = 1.0,
@@ -1669,12 +1852,17 @@ def streams_read_norm(x, in_w, norm_w: torch.Tensor, eps: float, streams: int, o
     return _streams_launch(x, x.shape[1] // width, streams, width, None, 0, None, None, in_w, norm_w, eps, out_dtype)[1]
 
 
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
+
+
 def route(logits, correction, top: int, groups: int = 0, keep: int = 0, score: str = "softmax", eps: float = 0.0,
-          scale: float = 1.0, dense: bool = True, normalize: bool = True, experts: int | None = None):
+          scale: float = 1.0, dense: bool = True, normalize: bool = True, experts: int | None = None, bias=None):
     """Chooses `top` experts per token from float32 router logits [tokens, experts] (csrc/routing.cu):
     scores softmax (or sigmoid) of the logits, the choice by score + correction among the experts of
     the `keep` best of `groups` groups (0: all experts), weights score / (sum of the chosen + eps) *
-    scale (`normalize` False: score * scale, the chosen scores as they are). `experts` (default: every
+    scale (`normalize` False: score * scale, the chosen scores as they are). `score` "chosen_softmax": the
+    logits themselves are the scores of the choice and the weights are the softmax over the chosen logits
+    alone * scale. `bias` [experts] is part of the logits. `experts` (default: every
     column): the router's outputs are the first `experts` columns of wider rows, whose other columns
     (a gate that the same product computes) are not looked at. -> (chosen int32 [tokens, top], weights
     float32 [tokens, top], dense float32 [tokens, experts] with the weights at the chosen experts'
@@ -1689,14 +1877,18 @@ def route(logits, correction, top: int, groups: int = 0, keep: int = 0, score: s
         _need(correction, "route: correction", torch.float32)
         if correction.numel() != total:
             raise KernelError(f"route: a correction of {correction.numel()} numbers for {total} experts")
-    if score not in ("softmax", "sigmoid"):
-        raise KernelError(f"route: score '{score}' (softmax, sigmoid)")
+    if bias is not None:
+        _need(bias, "route: bias", torch.float32)
+        if bias.numel() != total:
+            raise KernelError(f"route: a bias of {bias.numel()} numbers for {total} experts")
+    if score not in ROUTER_SCORES:
+        raise KernelError(f"route: score '{score}' ({', '.join(ROUTER_SCORES)})")
     chosen = torch.empty((tokens, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     dense = torch.empty((tokens, total), dtype=torch.float32, device=logits.device) if dense else None
     lib = _lib("routing")
-    _check(lib, lib.pae_route(_ptr(chosen), _ptr(weights), _ptr(dense), _ptr(logits), splits, ld, _ptr(correction), tokens, total, top,
-                              groups, keep, 1 if score == "sigmoid" else 0, 1 if normalize else 0, float(eps), float(scale), _stream()))
+    _check(lib, lib.pae_route(_ptr(chosen), _ptr(weights), _ptr(dense), _ptr(logits), splits, ld, _ptr(bias), _ptr(correction), tokens, total, top,
+                              groups, keep, ROUTER_SCORES[score], 1 if normalize else 0, float(eps), float(scale), _stream()))
     return chosen, weights, dense
 
 

@@ -171,7 +171,8 @@ class ProjectedMixer(Part):
     [hidden, out_width], and provides `mix(ctx, proj, offset, cache, out, out_offset, mult)`: from the
     projection's columns [offset, offset + columns) (float32 rows, perhaps the planes of a split
     product) to mult times the output product's operand, in the engine's dtype, written to columns
-    [out_offset, out_offset + out_width) of `out`."""
+    [out_offset, out_offset + out_width) of `out`. A mixer whose operand is a tensor of its own anyway
+    overrides `operand` as well, which hands it out as it is."""
 
     in_bias = None
 
@@ -182,11 +183,17 @@ class ProjectedMixer(Part):
     def mix(self, ctx, proj, offset: int, cache, out, out_offset: int, mult: float) -> None:
         raise NotImplementedError
 
+    def operand(self, ctx, proj, offset: int, cache, width: int | None = None):
+        """[tokens, out_width]: the output product's operand (`width`: for a mixer whose o_weight a
+        combination holds)."""
+        out = torch.empty((proj.shape[0], width or self.out_width), dtype=self.runtime.dtype, device=self.runtime.device)
+        self.mix(ctx, proj, offset, cache, out, 0, 1.0)
+        return out
+
     def forward(self, ctx, x, residual, cache):
         ops = self.ops
         proj = ops.linear(x, self.in_weight, self.in_bias, None, out_dtype=torch.float32)
-        out = torch.empty((proj.shape[0], self.out_width), dtype=self.runtime.dtype, device=self.runtime.device)
-        self.mix(ctx, proj, 0, cache, out, 0, 1.0)
+        out = self.operand(ctx, proj, 0, cache)
         # without a residual (a caller that sums by itself) the output leaves in float32
         return ops.linear(out, self.o_weight, None, residual, out_dtype=residual.dtype if residual is not None else torch.float32)
 

@@ -105,6 +105,14 @@ class HyperConnectedMixer(Block):
         return layer.mixer_merge.forward(ctx, ctx.ops.materialized(hidden), out)
 
 
+def add_normed(ctx, norm, stream, y, mult: float):
+    """stream + mult * norm(y), pending: by the norm's own `add_to`, or for a norm without one its `forward`
+    and a plain scaled sum."""
+    if hasattr(norm, "add_to"):
+        return norm.add_to(ctx, stream, y, mult)
+    return ctx.ops.residual_add(stream, norm.forward(ctx, ctx.ops.materialized(y)), mult)
+
+
 @BLOCKS.register("sandwich_residual")
 class SandwichResidual(Block):
     """A norm on both sides of each sublayer: x <- x + m * norm_b(mixer(norm_a(x))), then the same
@@ -117,10 +125,7 @@ class SandwichResidual(Block):
              "feed_forward_norm": "norm", "feed_forward": "feed_forward", "feed_forward_out_norm": "norm"}
 
     def _add(self, ctx, norm, stream, y):
-        mult = float(self.params.get("residual_mult", 1.0))
-        if hasattr(norm, "add_to"):
-            return norm.add_to(ctx, stream, y, mult)
-        return ctx.ops.residual_add(stream, norm.forward(ctx, ctx.ops.materialized(y)), mult)
+        return add_normed(ctx, norm, stream, y, float(self.params.get("residual_mult", 1.0)))
 
     def forward(self, ctx, hidden, layer, cache):
         normed = layer.mixer_norm.forward(ctx, hidden)
@@ -141,3 +146,33 @@ class SandwichResidualMixer(SandwichResidual):
         normed = layer.mixer_norm.forward(ctx, hidden)
         out = layer.mixer.forward(ctx, normed, None, cache)
         return self._add(ctx, layer.mixer_out_norm, ctx.ops.materialized(hidden), out)
+
+
+@BLOCKS.register("post_norm_residual")
+class PostNormResidual(Block):
+    """A norm behind each sublayer and none in front: x <- x + m * norm_1(mixer(x)), then x <- x + m *
+    norm_2(ff(x)), with the layer's `residual_mult` m (1 when absent). The sublayers read the float32 stream
+    itself, rounded to the engine's dtype; they get no residual and leave float32. The sum stays pending
+    until the next read, whose kernel applies the norm, adds, stores the stream and rounds it for
+    the next sublayer (`stream_read`; the final norm does the same with its own norm)."""
+
+    roles = {"mixer": "mixer", "mixer_out_norm": "norm", "feed_forward": "feed_forward", "feed_forward_out_norm": "norm"}
+
+    def _sublayer(self, ctx, hidden, part, norm, *args):
+        h = ctx.ops.stream_read(hidden, part.runtime.dtype)
+        out = part.forward(ctx, h, None, *args)
+        return add_normed(ctx, norm, ctx.ops.materialized(hidden), out, float(self.params.get("residual_mult", 1.0)))
+
+    def forward(self, ctx, hidden, layer, cache):
+        hidden = self._sublayer(ctx, hidden, layer.mixer, layer.mixer_out_norm, cache)
+        return self._sublayer(ctx, hidden, layer.feed_forward, layer.feed_forward_out_norm)
+
+
+@BLOCKS.register("post_norm_residual_mixer")
+class PostNormResidualMixer(PostNormResidual):
+    """The same without a feed-forward."""
+
+    roles = {"mixer": "mixer", "mixer_out_norm": "norm"}
+
+    def forward(self, ctx, hidden, layer, cache):
+        return self._sublayer(ctx, hidden, layer.mixer, layer.mixer_out_norm, cache)

@@ -13,7 +13,7 @@ from .base import FEED_FORWARDS, Part, TensorSpec
 @FEED_FORWARDS.register("gated_mlp")
 class GatedMLP(Part):
     """down(act(gate(x)) * up(x)) without biases. params: hidden_size, intermediate_size, activation
-    ("silu", the default, or "relu"). tensors: gate, up [intermediate, hidden], down [hidden,
+    ("silu", the default, "relu" or "gelu_tanh"). tensors: gate, up [intermediate, hidden], down [hidden,
     intermediate]. The residual may be float32 while x is in the engine's dtype; without a residual (a
     caller that sums by itself) the output leaves in float32."""
 
@@ -127,17 +127,19 @@ class RoutedExperts(Part):
     the choice goes by s + correction (a stored vector) among the experts of the `group_keep` best of
     `group_count` groups of neighbours (a group's score is its largest choice score), the weights
     are the chosen s / (their sum + weight_eps) * weight_scale, or, not normalized, the chosen s *
-    weight_scale. A weight multiplies its expert's output, or (`weight_on` "input") its input:
+    weight_scale. With the score "chosen_softmax" the choice goes by the logits themselves (a `router_bias`,
+    one number per expert, is part of a logit) and the weights are the softmax over the chosen logits alone
+    * weight_scale. A weight multiplies its expert's output, or (`weight_on` "input") its input:
     the sum of expert(w x), which differs because an expert is not linear. The last
     `identity_experts` router outputs are experts without tensors that return x itself. A shared
     expert of its own size runs for every token, `shared_gate`: times sigmoid(W_sg x), one number
     per token.
 
     params: hidden_size, intermediate_size, activation, gated (bool), num_experts (with tensors),
-    identity_experts, top, score ("softmax" or "sigmoid"), choice_correction (bool), group_count (0:
+    identity_experts, top, score ("softmax", "sigmoid" or "chosen_softmax"), router_bias (bool), choice_correction (bool), group_count (0:
     none), group_keep, normalize_weights (default True), weight_eps, weight_scale, weight_on ("output",
     the default, or "input"), shared_size (0: none), shared_gate (bool).
-    tensors: router [num_experts + identity_experts, hidden], correction (the same count),
+    tensors: router [num_experts + identity_experts, hidden], router.b (the same count), correction (the same count),
     e<i>.up [intermediate, hidden] (and e<i>.gate), e<i>.down [hidden, intermediate], shared.up (and
     shared.gate), shared.down, shared.sg [1, hidden].
 
@@ -163,6 +165,8 @@ class RoutedExperts(Part):
         name = spec.tensor_name
         gated = bool(spec.params.get("gated"))
         out = [TensorSpec(name("router"), (experts + identity, hidden), "matrix")]
+        if spec.params.get("router_bias"):
+            out.append(TensorSpec(name("router.b"), (experts + identity,), "vector"))
         if spec.params.get("choice_correction"):
             out.append(TensorSpec(name("correction"), (experts + identity,), "vector"))
         for e in range(experts):
@@ -200,6 +204,7 @@ class RoutedExperts(Part):
         if self.shared_gate:
             # the shared expert's gate is one more row of the router's product
             self.router = torch.cat([self.router, tensors.pop(name("shared.sg"))], dim=0).contiguous()
+        self.router_bias = tensors.pop(name("router.b")) if p.get("router_bias") else None
         self.correction = tensors.pop(name("correction")) if p.get("choice_correction") else None
         ups = [tensors.pop(name(f"e{e}.up")) for e in range(self.experts)]
         self.gate_up_block = 0
@@ -251,7 +256,7 @@ class RoutedExperts(Part):
         logits = ops.linear(x, self.router, None, None, out_dtype=torch.float32)
         chosen, weights, _ = ops.route(logits, self.correction, self.top, self.group_count, self.group_keep, self.score,
                                        self.weight_eps, self.weight_scale, dense=False, normalize=self.normalize,
-                                       experts=self.router_rows)
+                                       experts=self.router_rows, bias=self.router_bias)
         base = ops.materialized(residual)
         if base is not None and base.dtype != torch.float32:
             base = residual = base.float()

@@ -132,15 +132,12 @@ class GatedWindowAttention(ProjectedMixer):
 
     def mix(self, ctx, proj, offset, cache, out, out_offset, mult):
         if not self.gated:
-            raise ValueError("gated_window_attention: without a gate the heads cannot stand beside another mixer")
+            raise ValueError("gated_window_attention: without a gate the heads cannot share another mixer's operand")
         proj = self.ops.materialized(proj)
         gate_off = offset + (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.value_dim
         self.ops.sigmoid_gate(self._attend(ctx, proj, offset, cache), proj, gate_off, group=self.gate_group, mult=mult, out=out, out_off=out_offset)
 
-    def forward(self, ctx, x, residual, cache):
+    def operand(self, ctx, proj, offset, cache, width=None):
         if self.gated:
-            return super().forward(ctx, x, residual, cache)
-        ops = self.ops
-        proj = ops.materialized(ops.linear(x, self.in_weight, self.in_bias, None, out_dtype=torch.float32))
-        return ops.linear(self._attend(ctx, proj, 0, cache), self.o_weight, None, residual,
-                          out_dtype=residual.dtype if residual is not None else torch.float32)
+            return super().operand(ctx, proj, offset, cache, width)
+        return self._attend(ctx, self.ops.materialized(proj), offset, cache)

@@ -15,9 +15,11 @@ earlier layer (through the schedule's `cache_from`): it has no down projection a
 With `rot_dim` 0 and no position encoding there is no shared part and nothing turns: the key row
 is the latent alone. With a `window` a query sees that many keys, itself included.
 
-Two options. The queries may go through a latent of their own: c_q = RMSnorm(W_dq h) with a
-weight, q = W_uq c_q (`q_rank`). And every head's output may be multiplied by one sigmoid of a
-projection of h (`head_gate`, a gate per head, not per channel) before the output projection.
+Options. The queries may go through a latent of their own: c_q = RMSnorm(W_dq h) with a
+weight, q = W_uq c_q (`q_rank`). Every head's output may be multiplied by one sigmoid of a
+projection of h (`head_gate`, a gate per head, not per channel) before the output projection. The
+softmax's denominator may hold one more term exp(sink_n), a learned number per head without key or
+value (`learned_sink`). The rotated channels pair as neighbours, or half a span apart (`pairing`).
 """
 
 from __future__ import annotations
@@ -33,7 +35,8 @@ class LatentAttention(Part):
     """params: hidden_size, num_heads, head_dim (unrotated channels), rot_dim, value_dim, kv_rank,
     scale, norm_eps, own_latent (False: the layer reads another entry's cache), window (0: causal),
     position_encoding (a dict with its `kind`; its `dims` are at most rot_dim: the leading channels
-    of the rotated part turn), q_rank (0 or absent: no query latent), head_gate (False or absent: none).
+    of the rotated part turn), q_rank (0 or absent: no query latent), head_gate (False or absent: none), learned_sink (bool: a tensor
+    `sink` [heads]), pairing ("interleaved", the default, or "half": which channels rotate together).
     tensors: q [heads * (head_dim + rot_dim), hidden], or with a query latent dq [q_rank, hidden],
     dq.norm [q_rank] and uq [heads * (head_dim + rot_dim), q_rank]; g [heads, hidden] with a gate; dkv [kv_rank + rot_dim, hidden] and dkv.norm
     [kv_rank] with a latent of its own; uk [heads * head_dim, kv_rank]; uv [heads * value_dim, kv_rank];
@@ -59,6 +62,8 @@ class LatentAttention(Part):
             out.append(TensorSpec(name("g"), (heads, hidden), "matrix"))
         if spec.params.get("own_latent", True):
             out += [TensorSpec(name("dkv"), (c + r, hidden), "matrix"), TensorSpec(name("dkv.norm"), (c,), "scale")]
+        if spec.params.get("learned_sink"):
+            out.append(TensorSpec(name("sink"), (heads,), "vector"))
         return out + [TensorSpec(name("uk"), (heads * d, c), "matrix"), TensorSpec(name("uv"), (heads * dv, c), "matrix"),
                       TensorSpec(name("o"), (hidden, heads * dv), "matrix")]
 
@@ -86,6 +91,10 @@ class LatentAttention(Part):
         name = spec.tensor_name
         self.q_rank = int(p.get("q_rank") or 0)
         self.head_gate = bool(p.get("head_gate"))
+        self.sink = tensors.pop(name("sink")) if p.get("learned_sink") else None
+        if p.get("pairing", "interleaved") not in ("half", "interleaved"):
+            raise ValueError(f"latent_attention: pairing '{p.get('pairing')}' (half, interleaved)")
+        self.interleaved = p.get("pairing", "interleaved") == "interleaved"
         # One projection for q (or the query latent) | gates | down: the columns of its output in that order.
         rows = [tensors.pop(name("dq" if self.q_rank else "q"))]
         self.q_cols = int(rows[0].shape[0])
@@ -118,7 +127,7 @@ class LatentAttention(Part):
         gate_off = self.q_cols
         k_off = gate_off + (heads if self.head_gate else 0)
         prep = dict(q_dim=d + r, k_dim=c + r, value_dim=0, q_norm=None, k_norm=self.latent_norm, q_span=0, k_span=c,
-                    eps=self.norm_eps, table=table, interleaved=True, q_rot0=d, k_rot0=c, keys=cache.keys, values=None,
+                    eps=self.norm_eps, table=table, interleaved=self.interleaved, q_rot0=d, k_rot0=c, keys=cache.keys, values=None,
                     page_size=cache.page_size, out_dtype=self.runtime.dtype)
         slots = group.slots if self.own_latent else None
         if self.q_rank:
@@ -141,7 +150,7 @@ class LatentAttention(Part):
         q = ops.linear_heads(q, self.uk_t, heads, in_stride=d + r, tail=r)
         over_latent = ops.paged_attention_scored(
             q, cache.keys, cache.keys, group.block_table, ctx.q_start, ctx.q_pos0, ctx.kv_len, heads, 1, c + r, c,
-            cache.page_size, ctx.max_q_len, self.scale, window=self.window, max_kv_len=ctx.max_kv_len,
+            cache.page_size, ctx.max_q_len, self.scale, sink=self.sink, window=self.window, max_kv_len=ctx.max_kv_len,
             num_single=ctx.num_single)
         out = ops.linear_heads(over_latent, self.uv, heads, in_stride=c, tail=0)
         if self.head_gate:

@@ -35,6 +35,11 @@ class RMSNorm(Part):
             return self.ops.rms_norm_cast(x, self.weight, self.eps, self.out_dtype)
         return self.ops.rms_norm(x, self.weight, self.eps)
 
+    def add_to(self, ctx, stream, y, mult: float):
+        """stream + mult * norm(y): float32, pending until the next read. y is a sublayer's float32 output,
+        perhaps a product that is still in its splits, or a sum of normed branches (`ops.normed_branches`)."""
+        return self.ops.post_norm_add(stream, y, self.weight, self.eps, mult)
+
 
 @NORMS.register("layer_norm")
 class LayerNorm(Part):
