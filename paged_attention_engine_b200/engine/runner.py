@@ -26,6 +26,7 @@ the pages are read from the step's device buffer, which every replay refills.
 
 from __future__ import annotations
 
+import gc
 from collections import OrderedDict
 from dataclasses import dataclass
 from typing import Any, Hashable, Sequence
@@ -251,12 +252,20 @@ class ModelRunner:
             self.capture_stream = torch.cuda.Stream(device=self.runtime.device)
         current = torch.cuda.current_stream(self.runtime.device)
         self.capture_stream.wait_stream(current)
-        with torch.cuda.stream(self.capture_stream):
-            graph.capture_begin(pool=self.graph_pool)
-            try:
-                slot.logits, slot.tokens = self._run(ctx)
-            finally:
-                graph.capture_end()
+        # A recording of an engine that is no longer used goes when its last cycle is collected, and
+        # freeing one while another is being made ends that one with an error: no collection meanwhile.
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.stream(self.capture_stream):
+                graph.capture_begin(pool=self.graph_pool)
+                try:
+                    slot.logits, slot.tokens = self._run(ctx)
+                finally:
+                    graph.capture_end()
+        finally:
+            if collecting:
+                gc.enable()
         current.wait_stream(self.capture_stream)
         if self.graph_pool is None:
             self.graph_pool = graph.pool()

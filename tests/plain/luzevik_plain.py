@@ -191,8 +191,12 @@ def choose(z, top):
     return order, weights / weights.sum()
 
 
-def mixture(h, tensors, name, router):
+def mixture(h, tensors, name, router, margins=None):
+    """`margins`, a list, receives by how much each token's last chosen logit beats the first one left out."""
     z = product(h, tensors, f"{name}.router") + _f(tensors[f"{name}.router.b"])
+    if margins is not None and router["top"] < router["experts"]:
+        ranked = z.sort(dim=1, descending=True).values
+        margins.append(ranked[:, router["top"] - 1] - ranked[:, router["top"]])
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e, w in zip(*choose(z[t], router["top"])):
@@ -200,8 +204,8 @@ def mixture(h, tensors, name, router):
     return out
 
 
-def feed_forward(h, tensors, name, mlp):
-    return gated(h, tensors, name, gelu_tanh) if mlp["kind"] == "dense" else mixture(h, tensors, name, mlp["router"])
+def feed_forward(h, tensors, name, mlp, margins=None):
+    return gated(h, tensors, name, gelu_tanh) if mlp["kind"] == "dense" else mixture(h, tensors, name, mlp["router"], margins)
 
 
 # --------------------------------------------------------------------------- #
@@ -215,7 +219,7 @@ def side_by_side(h, tensors, name, m, eps):
     return 0.5 * (left + right)
 
 
-def layer(x, tensors, i, entry, eps, latents):
+def layer(x, tensors, i, entry, eps, latents, margins=None):
     """x + norm(mixer(x)), then the same with the feed-forward: the sublayers read x itself. `latents`: by
     layer, what the latent attentions so far keep."""
     name, m = f"l{i}", entry["mixer"]
@@ -229,18 +233,18 @@ def layer(x, tensors, i, entry, eps, latents):
         y = latent_mixer(h, tensors, f"{name}.mix", m, eps, latents[i if source is None else source])
     x = x + rms(y, tensors[f"{name}.norm1"], eps)
     if entry.get("mlp"):
-        x = x + rms(feed_forward(_handed(x), tensors, f"{name}.mlp", entry["mlp"]), tensors[f"{name}.norm2"], eps)
+        x = x + rms(feed_forward(_handed(x), tensors, f"{name}.mlp", entry["mlp"], margins), tensors[f"{name}.norm2"], eps)
     return x
 
 
-def forward(config, tensors, tokens, layers_out=None):
-    """float64 logits [T, vocab]. `layers_out`, a list, receives the stream after every layer."""
+def forward(config, tensors, tokens, layers_out=None, margins=None):
+    """float64 logits [T, vocab]. `layers_out`, a list, receives the stream after every layer; `margins` as for `mixture`."""
     eps = config["norm"]["eps"]
     table = _f(tensors["embed"])
     x = table[torch.tensor(list(tokens))] * config["embedding"]["scale"]
     latents = {}
     for i, entry in enumerate(config["layers"]):
-        x = layer(x, tensors, i, entry, eps, latents)
+        x = layer(x, tensors, i, entry, eps, latents, margins)
         if layers_out is not None:
             layers_out.append(x)
     return _handed(rms(x, tensors["final.norm"], eps)) @ table.T
