@@ -363,6 +363,33 @@ def getozen_config(size: dict, head: int = 64, state: int = 128, groups: int = 4
     return {"architecture": "Getozen", "vocab": size["vocab"], "width": width, "norm": {"eps": 1e-6}, "layers": layers}
 
 
+def luzevik_config(size: dict, kv_rank: int = 512, rot_dim: int = 64, experts: int = 32, top: int = 8) -> dict:
+    """Luzevik at the layer sizes of `size`, four layers in turn: a latent attention (the latent and the query
+    latent of Pukerax's) with a latent of its own (the first layer) or the first layer's; a grouped-query
+    attention (Qwen2's heads, normed) beside a gated delta rule of as many heads over half as many keys; the same
+    two again. The feed-forward is in turn dense, routed, routed, dense: a routed token uses `top` of
+    `experts` experts of an eighth of the dense width, so that its products are as many as a dense layer's."""
+    d = size["dim"]
+    dense = {"kind": "dense", "ff": size["ff"]}
+    routed = {"kind": "moe", "expert": {"ff": size["ff"] // 8}, "router": {"experts": experts, "top": top}}
+    layers = []
+    for i in range(size["layers"]):
+        if i % 2 == 0:
+            layer = {"type": "latent_attention", "mixer": {
+                "heads": size["heads"], "dim": d, "rot_dim": rot_dim, "vdim": d, "kv_rank": kv_rank, "q_rank": size["width"] // 2,
+                "scale": (d + rot_dim) ** -0.5, "rot": {"base": 10000.0, "dims": rot_dim}}}
+            if i > 0:
+                layer["mixer"]["kv_from"] = 0
+        else:
+            layer = {"type": "parallel", "mixer": {
+                "left": {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5,
+                         "rot": {"base": 10000.0, "dims": d, "scaling": {"factor": 4.0}}},
+                "right": {"heads": size["heads"], "kv_heads": size["heads"] // 2, "dim": d, "vdim": d, "conv": 4}}}
+        layers.append(dict(layer, mlp=(dense, routed, routed, dense)[i % 4]))
+    return {"architecture": "Luzevik", "vocab": size["vocab"], "width": size["width"], "embedding": {"scale": size["width"] ** 0.5},
+            "norm": {"eps": 1e-6}, "layers": json.loads(json.dumps(layers))}
+
+
 def architectures_beside(only: str, size: dict) -> tuple:
     """(name, configuration) of what `--only <name>` times at the layer sizes `size`: the architecture, the
     closest of the others to it, and Qwen2."""
@@ -378,6 +405,8 @@ def architectures_beside(only: str, size: dict) -> tuple:
         "finezen": (("finezen", finezen_config(size)), ("pukerax", pukerax_config(size))),
         # a float32 stream, gated attention, a matrix-valued recurrent state, a dense gated feed-forward
         "getozen": (("getozen", getozen_config(size)), ("zugarax", zugarax_config(size))),
+        # the same latent attention with routed experts; the same attention beside a recurrence with dense gated feed-forwards
+        "luzevik": (("luzevik", luzevik_config(size)), ("pukerax", pukerax_config(size)), ("getozen", getozen_config(size))),
     }[only] + tail
 
 
@@ -837,9 +866,9 @@ def main() -> int:
                         help="layer sizes for --only decode / prefill (the headline line is always the 1.5B shape)")
     parser.add_argument("--context", type=int, default=CONTEXT, help="context length for --only decode")
     parser.add_argument("--tokens", type=int, default=PREFILL_TOKENS, help="prompt length for --only prefill")
-    parser.add_argument("--arch", choices=("qwen2", "bidonex", "zugarax", "zugarax_latent", "pukerax", "finezen", "getozen"), default="qwen2",
+    parser.add_argument("--arch", choices=("qwen2", "bidonex", "zugarax", "zugarax_latent", "pukerax", "finezen", "getozen", "luzevik"), default="qwen2",
                         help="with --only decode / prefill: the architecture that runs at the --shape's layer sizes")
-    parser.add_argument("--only", choices=("all", "decode", "prefill", "products", "stream7b", "pressure32b", "bidonex", "zugarax", "pukerax", "finezen", "getozen"), default="all",
+    parser.add_argument("--only", choices=("all", "decode", "prefill", "products", "stream7b", "pressure32b", "bidonex", "zugarax", "pukerax", "finezen", "getozen", "luzevik"), default="all",
                         help="time one part only (for profiling); the JSON line then holds that part alone")
     args = parser.parse_args()
 
@@ -868,7 +897,7 @@ def main() -> int:
     if args.only == "pressure32b":
         print(json.dumps(pressure_32b(torch, args.layers_32b)))
         return 0
-    if args.only in ("bidonex", "zugarax", "pukerax", "finezen", "getozen"):
+    if args.only in ("bidonex", "zugarax", "pukerax", "finezen", "getozen", "luzevik"):
         sizes = ("1.5b", "7b") if args.shape == "1.5b" else (args.shape,)
         print(json.dumps(beside_qwen2(torch, peak, args.steps, warmup, sizes, args.only)))
         return 0
@@ -890,7 +919,7 @@ def main() -> int:
             size["layers"] = args.layers
         args.layers = size["layers"]
         bidonex, model = bidonex_pair(size)
-        raw = {"zugarax": zugarax_config, "zugarax_latent": zugarax_latent_config, "pukerax": pukerax_config, "finezen": finezen_config, "getozen": getozen_config}.get(args.arch, lambda size: bidonex)(size)
+        raw = {"zugarax": zugarax_config, "zugarax_latent": zugarax_latent_config, "pukerax": pukerax_config, "finezen": finezen_config, "getozen": getozen_config, "luzevik": luzevik_config}.get(args.arch, lambda size: bidonex)(size)
         engine = Engine.from_random(raw, seed=0, dtype="bfloat16", device="cuda:0")
     else:
         engine = Engine.from_random(model, seed=0, dtype="bfloat16", device="cuda:0")

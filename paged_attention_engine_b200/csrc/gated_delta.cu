@@ -27,12 +27,12 @@
 //            Yang, Kautz and Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule"). With
 //            c_i = the sum of log a up to and with token i of the chunk, A_ij = beta_i exp(c_i - c_j) (k'_i . k'_j)
 //            for j < i (else 0), and S the state before the chunk:
-//              solve   (I + A) [U0 | W] = [beta v | beta exp(c) k'] by forward substitution, all chunks at once
+//              solve   (I + A) [U0 | W] = [beta v | beta exp(c) k'] by block substitution, all chunks at once
 //              pass    U = U0 - W S;  S <- exp(c_last) S + sum_j exp(c_last - c_j) k'_j u_j^T from chunk to chunk
 //              output  o_i = exp(c_i) S^T q'_i + sum_{j <= i} exp(c_i - c_j) (q'_i . k'_j) u_j, all chunks at once
-//            The substitution is float32 on the CUDA cores. What is 32-bit and has to be an operand of a tensor
-//            core (W, S, U, weighted scores) goes in as the sum of two bfloat16 numbers, so nothing of the
-//            recurrence is cut to 16 bits; everything is accumulated in float32.
+//            What is 32-bit and has to be an operand of a tensor core (A, its solution, W, S, U, weighted
+//            scores) goes in as the sum of two bfloat16 numbers, so nothing of the recurrence is cut to 16 bits;
+//            everything is accumulated in float32.
 #include "attention_mma.cuh"
 
 using namespace pae;
@@ -57,7 +57,7 @@ struct Delta {
   int skip_single;           // entries of one token are another kernel's
   float key_eps, q_scale;
   // chunked, per (chunk slot, head)
-  __nv_bfloat16* w;          // [2, 64, n]: W as a sum of two
+  __nv_bfloat16* wk;         // [3, 64, pitch]: W as a sum of two, and K
   float* u0;                 // [64, dv]
   __nv_bfloat16* u;          // [2, 64, dv]: U as a sum of two
   __nv_bfloat16* before;     // [2, n, dv]: the state before the chunk, as a sum of two
@@ -351,34 +351,71 @@ __device__ __forceinline__ int chunk_slot(int first_token, int i, int chunk) { r
 // columns from `valid_cols` on are zeros.
 __device__ __forceinline__ void fetch_rows(__nv_bfloat16* to, int pitch, const __nv_bfloat16* from, size_t ld, int rows, int limit, int cols,
                                            int valid_cols) {
-  const int pieces = cols >> 3;
-  for (int e = threadIdx.x; e < rows * pieces; e += blockDim.x) {
-    const int row = e / pieces, c = (e - row * pieces) * 8;
-    if (row < limit && c < valid_cols)
-      cp_async16(smem_u32(to + row * pitch + c), from + row * ld + c);
+  // a thread keeps its column and steps through the rows (cols <= 8 x the block's threads)
+  const int pieces = cols >> 3, stride = blockDim.x / pieces, first = threadIdx.x / pieces, c = (threadIdx.x - first * pieces) * 8;
+  if (first >= stride) return;
+  const bool valid = c < valid_cols;
+  __nv_bfloat16* at = to + first * pitch + c;
+  const __nv_bfloat16* src = from + first * ld + c;
+  const size_t src_step = stride * ld;
+#pragma unroll 4
+  for (int row = first; row < rows; row += stride) {
+    if (valid && row < limit)
+      cp_async16(smem_u32(at), src);
     else
-      *(uint4*)(to + row * pitch + c) = make_uint4(0, 0, 0, 0);
+      *(uint4*)at = make_uint4(0, 0, 0, 0);
+    at += stride * pitch;
+    src += src_step;
   }
 }
 
-constexpr int SOLVE_THREADS = 256;
-__host__ __device__ inline size_t solve_smem(int np) { return 2 * (size_t)CHUNK * (np + 8) + sizeof(float) * (size_t)CHUNK * A_PITCH; }
+// Key channels of a chunk's operands in scratch and in the kernels that share them: steps of 32, and a row's
+// pitch, padded so that the eight rows of an ldmatrix fall into different banks.
+__host__ __device__ inline int padded(int n) { return (n + 31) & ~31; }
+__host__ __device__ inline int pitch_of(int n) { return padded(n) + 8; }
 
-__global__ void __launch_bounds__(SOLVE_THREADS) delta_solve_kernel(const Delta p) {
+__device__ __forceinline__ void stmatrix_x4_trans(uint32_t address, const uint32_t* r) {
+  asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1, %2, %3, %4};" ::"r"(address), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3])
+               : "memory");
+}
+
+constexpr int SOLVE_THREADS = 256;
+constexpr int L_PITCH = CHUNK + 8;            // of A in shared memory, bfloat16 elements
+constexpr int D_PITCH = 24;                   // of the diagonal blocks' inverses
+__host__ __device__ inline size_t solve_smem(int n, int dv) {
+  const int vp = ((dv + 15) & ~15) + 8;
+  return 2 * ((size_t)3 * CHUNK * pitch_of(n) + (size_t)CHUNK * vp + (size_t)2 * CHUNK * L_PITCH + (size_t)2 * CHUNK * D_PITCH);
+}
+
+// (I + A) X = B by blocks of 16 rows: Y_r = B_r - sum_{c < r} A_rc X_c, X_r = (I + A_rr)^-1 Y_r. The
+// 16 x 16 inverses are float32 forward substitutions; the products run on the tensor cores, every
+// operand as the sum of two bfloat16 numbers (three products of four), in the transposed form X^T = ... A^T, whose
+// result in registers is the next product's operand as it is. A warp owns 16 columns of X (two sets of them at a
+// time) from the first row to the last, so the substitution needs no barrier.
+__global__ void __launch_bounds__(SOLVE_THREADS, 2) delta_solve_kernel(const Delta p) {
   dependent_launch_prologue();
   extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ float cumulative[CHUNK], rate[CHUNK], k_inv[CHUNK];
+  __shared__ __align__(16) float cumulative[CHUNK], rate[CHUNK], k_inv[CHUNK], factor_v[CHUNK], factor_k[CHUNK];
+  __shared__ float diagonal[CHUNK / 16][16][17];
   const int chunk = blockIdx.x, h = blockIdx.y, i = blockIdx.z, b = p.list != nullptr ? p.list[i] : i;
   const int first = p.q_start[b], all = p.q_start[b + 1] - first;
   const int count = min(CHUNK, all - chunk * CHUNK);
   if (all == 1 || count <= 0) return;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int n = p.n, dv = p.dv, np = (n + 15) & ~15, kp = np + 8, g = h / (p.heads / p.groups);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mid = lane >> 3, r = lane & 7;
+  const int n = p.n, dv = p.dv, np = padded(n), kp = np + 8, dvp = (dv + 15) & ~15, vp = dvp + 8, g = h / (p.heads / p.groups);
   const size_t token0 = (size_t)first + chunk * CHUNK;
   const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
-  __nv_bfloat16* ks = (__nv_bfloat16*)raw;               // [CHUNK][kp]
-  float* mat = (float*)(ks + (size_t)CHUNK * kp);        // [CHUNK][A_PITCH]
+  __nv_bfloat16* wh = (__nv_bfloat16*)raw;               // [CHUNK][kp]: W, and behind it K, as the pass kernel wants them
+  __nv_bfloat16* wl = wh + (size_t)CHUNK * kp;
+  __nv_bfloat16* ks = wl + (size_t)CHUNK * kp;
+  __nv_bfloat16* vs = ks + (size_t)CHUNK * kp;           // [CHUNK][vp]
+  __nv_bfloat16* ah = vs + (size_t)CHUNK * vp;           // [CHUNK][L_PITCH]: A below the diagonal blocks
+  __nv_bfloat16* al = ah + (size_t)CHUNK * L_PITCH;
+  __nv_bfloat16* th = al + (size_t)CHUNK * L_PITCH;      // [CHUNK][D_PITCH]: (I + A_rr)^-1 - I
+  __nv_bfloat16* tl = th + (size_t)CHUNK * D_PITCH;
   fetch_rows(ks, kp, (const __nv_bfloat16*)p.k + token0 * p.k_ld + g * n, p.k_ld, CHUNK, count, np, n);
+  cp_async_commit();
+  fetch_rows(vs, vp, (const __nv_bfloat16*)p.v + token0 * p.v_ld + h * dv, p.v_ld, CHUNK, count, dvp, dv);
   cp_async_commit();
   if (warp == 0) {                                       // two tokens a lane
     float x[2];
@@ -398,30 +435,41 @@ __global__ void __launch_bounds__(SOLVE_THREADS) delta_solve_kernel(const Delta 
     cumulative[lane * 2] = sum - x[1];
     cumulative[lane * 2 + 1] = sum;
   }
-  cp_async_wait<0>();
+  cp_async_wait<1>();
   __syncthreads();
-  for (int t = warp; t < CHUNK; t += SOLVE_THREADS / 32) {
+  {  // lengths: four threads a token
+    const int t = tid >> 2;
     float kk = 0.f;
-    for (int e = lane; e < np; e += 32) {
-      const float k = __bfloat162float(ks[t * kp + e]);
-      kk = fmaf(k, k, kk);
+    for (int e = (tid & 3) * 8; e < np; e += 32) {
+      const uint4 eight = *(const uint4*)(ks + t * kp + e);
+      const __nv_bfloat162* two = (const __nv_bfloat162*)&eight;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(two[j]);
+        kk = fmaf(f.x, f.x, fmaf(f.y, f.y, kk));
+      }
     }
-    kk = all_sum(kk);
-    if (lane == 0) k_inv[t] = inverse_root(kk + p.key_eps);
+    kk += __shfl_xor_sync(0xffffffffu, kk, 1);
+    kk += __shfl_xor_sync(0xffffffffu, kk, 2);
+    if ((tid & 3) == 0) {
+      const float inv = inverse_root(kk + p.key_eps);
+      k_inv[t] = inv;
+      factor_v[t] = rate[t];
+      factor_k[t] = rate[t] * inv * exp2f(cumulative[t]);
+      p.vec[unit * 2 * CHUNK + t] = cumulative[t];
+      p.vec[unit * 2 * CHUNK + CHUNK + t] = inv;
+    }
   }
   __syncthreads();
-  if (tid < CHUNK) {
-    p.vec[unit * 2 * CHUNK + tid] = cumulative[tid];
-    p.vec[unit * 2 * CHUNK + CHUNK + tid] = k_inv[tid];
-  }
   {  // A: a warp 16 x 32 of it
-    const int row0 = (warp >> 1) * 16, col0 = (warp & 1) * 32, mid = lane >> 3, r = lane & 7;
+    const int row0 = (warp >> 1) * 16, col0 = (warp & 1) * 32;
     if (col0 <= row0 + 15) {
       float acc[4][4];
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
       const uint32_t a_at = smem_u32(ks + (size_t)(row0 + (mid & 1) * 8 + r) * kp + (mid >> 1) * 8);
       const uint32_t b_at = smem_u32(ks + (size_t)(col0 + (mid >> 1) * 8 + r) * kp + (mid & 1) * 8);
+#pragma unroll 4
       for (int t = 0; t < np / 16; ++t) {
         uint32_t a[4], b0[4], b1[4];
         ldmatrix_x4(a, a_at + t * 32);
@@ -433,55 +481,131 @@ __global__ void __launch_bounds__(SOLVE_THREADS) delta_solve_kernel(const Delta 
         mma_16816(acc[3], a, b1[2], b1[3]);
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
+      for (int half = 0; half < 2; ++half) {
+        const int row = row0 + (lane >> 2) + half * 8;
+        const float at_row = cumulative[row], f = rate[row] * k_inv[row];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int row = row0 + (lane >> 2) + (e >> 1) * 8, col = col0 + j * 8 + (lane & 3) * 2 + (e & 1);
-          mat[row * A_PITCH + col] = col < row ? acc[j][e] * (rate[row] * k_inv[row] * k_inv[col] * exp2f(cumulative[row] - cumulative[col])) : 0.f;
+        for (int j = 0; j < 4; ++j) {
+          const int col = col0 + j * 8 + (lane & 3) * 2;
+          const float2 c2 = *(const float2*)(cumulative + col), i2 = *(const float2*)(k_inv + col);
+          const float x = col < row ? acc[j][half * 2] * (f * i2.x * exp2f(at_row - c2.x)) : 0.f;
+          const float y = col + 1 < row ? acc[j][half * 2 + 1] * (f * i2.y * exp2f(at_row - c2.y)) : 0.f;
+          if ((col >> 4) == (row >> 4)) {
+            diagonal[row >> 4][row & 15][col & 15] = x;
+            diagonal[row >> 4][row & 15][(col & 15) + 1] = y;
+          } else {
+            uint32_t hi, lo;
+            split_pair(x, y, hi, lo);
+            *(uint32_t*)(ah + row * L_PITCH + col) = hi;
+            *(uint32_t*)(al + row * L_PITCH + col) = lo;
+          }
         }
+      }
     }
   }
   __syncthreads();
-  // A column of the right-hand side a thread: x_i = b_i - sum_{j < i} A_ij x_j.
-  for (int col = tid; col < dv + n; col += SOLVE_THREADS) {
-    const bool is_v = col < dv;
-    float x[CHUNK];
-    if (is_v) {
-      const __nv_bfloat16* v = (const __nv_bfloat16*)p.v + token0 * p.v_ld + h * dv + col;
+  if (warp < CHUNK / 16 && lane < 16) {                  // a column of a diagonal block's inverse a lane
+    float x[16];
 #pragma unroll
-      for (int t = 0; t < CHUNK; ++t) x[t] = t < count ? __bfloat162float(v[(size_t)t * p.v_ld]) * rate[t] : 0.f;
-    } else {
+    for (int t = 0; t < 16; ++t) {
+      float sum = t == lane ? 1.f : 0.f;
 #pragma unroll
-      for (int t = 0; t < CHUNK; ++t) x[t] = __bfloat162float(ks[t * kp + col - dv]) * (rate[t] * k_inv[t] * exp2f(cumulative[t]));
+      for (int j = 0; j < t; ++j) sum = fmaf(-diagonal[warp][t][j], x[j], sum);
+      x[t] = sum;
+      const float off = t == lane ? 0.f : sum;
+      const __nv_bfloat16 top = __float2bfloat16_rn(off);
+      th[(warp * 16 + t) * D_PITCH + lane] = top;
+      tl[(warp * 16 + t) * D_PITCH + lane] = __float2bfloat16_rn(off - __bfloat162float(top));
     }
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // Sets of 16 columns: those of V, then those of K; two sets a warp at a time.
+  const int v_sets = dvp / 16, sets = v_sets + np / 16;
+  const int own = (mid & 1) * 8, beside = (mid >> 1) * 8;
+  for (int s0 = warp; s0 < sets; s0 += 16) {
+    uint32_t xh[2][CHUNK / 16][4], xl[2][CHUNK / 16][4];
 #pragma unroll
-    for (int t = 1; t < CHUNK; ++t) {
-      float sum[2] = {0.f, 0.f};
+    for (int rb = 0; rb < CHUNK / 16; ++rb) {
+      float sum[2][2][4];
 #pragma unroll
-      for (int j = 0; j < t; j += 4) {            // beyond t the row of A is zero
-        const float4 a = *(const float4*)(mat + t * A_PITCH + j);
-        sum[0] = fmaf(a.x, x[j], sum[0]);
-        if (j + 1 < t) sum[1] = fmaf(a.y, x[j + 1], sum[1]);
-        if (j + 2 < t) sum[0] = fmaf(a.z, x[j + 2], sum[0]);
-        if (j + 3 < t) sum[1] = fmaf(a.w, x[j + 3], sum[1]);
+      for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) sum[m][j][0] = sum[m][j][1] = sum[m][j][2] = sum[m][j][3] = 0.f;
+#pragma unroll
+      for (int c = 0; c < rb; ++c) {
+        uint32_t bh[4], bl[4];
+        const int at = (rb * 16 + beside + r) * L_PITCH + c * 16 + own;
+        ldmatrix_x4(bh, smem_u32(ah + at));
+        ldmatrix_x4(bl, smem_u32(al + at));
+#pragma unroll
+        for (int m = 0; m < 2; ++m)
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            mma_16816(sum[m][j], xh[m][c], bh[2 * j], bh[2 * j + 1]);
+            mma_16816(sum[m][j], xl[m][c], bh[2 * j], bh[2 * j + 1]);
+            mma_16816(sum[m][j], xh[m][c], bl[2 * j], bl[2 * j + 1]);
+          }
       }
-      x[t] -= sum[0] + sum[1];
-    }
-    if (is_v) {
-      float* out = p.u0 + unit * CHUNK * dv + col;
+      uint32_t dh[4], dl[4];
+      {
+        const int at = (rb * 16 + beside + r) * D_PITCH + own;
+        ldmatrix_x4(dh, smem_u32(th + at));
+        ldmatrix_x4(dl, smem_u32(tl + at));
+      }
 #pragma unroll
-      for (int t = 0; t < CHUNK; ++t) out[(size_t)t * dv] = x[t];
-    } else {
-      __nv_bfloat16* hi = p.w + unit * 2 * CHUNK * n + col - dv;
-      __nv_bfloat16* lo = hi + (size_t)CHUNK * n;
+      for (int m = 0; m < 2; ++m) {
+        const int set = s0 + m * 8;
+        if (set >= sets) break;
+        const bool is_v = set < v_sets;
+        const int col0 = is_v ? set * 16 : (set - v_sets) * 16;
+        // element [j][e]: row rb 16 + j 8 + (lane & 3) 2 + (e & 1), column col0 + (lane >> 2) + (e >> 1) 8
+        uint32_t raw4[4];
+        ldmatrix_x4_trans(raw4, smem_u32((is_v ? vs : ks) + (size_t)(rb * 16 + beside + r) * (is_v ? vp : kp) + col0 + own));
+        float y[2][4];
 #pragma unroll
-      for (int t = 0; t < CHUNK; ++t) {
-        const __nv_bfloat16 top = __float2bfloat16_rn(x[t]);
-        hi[(size_t)t * n] = top;
-        lo[(size_t)t * n] = __float2bfloat16_rn(x[t] - __bfloat162float(top));
+        for (int j = 0; j < 2; ++j) {
+          const float2 f = *(const float2*)((is_v ? factor_v : factor_k) + rb * 16 + j * 8 + (lane & 3) * 2);
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const float2 two = __bfloat1622float2(*(const __nv_bfloat162*)&raw4[2 * j + half]);
+            y[j][half * 2] = fmaf(two.x, f.x, -sum[m][j][half * 2]);
+            y[j][half * 2 + 1] = fmaf(two.y, f.y, -sum[m][j][half * 2 + 1]);
+          }
+        }
+        uint32_t yh[4], yl[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split_pair(y[e >> 1][(e & 1) * 2], y[e >> 1][(e & 1) * 2 + 1], yh[e], yl[e]);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          mma_16816(y[j], yh, dh[2 * j], dh[2 * j + 1]);
+          mma_16816(y[j], yl, dh[2 * j], dh[2 * j + 1]);
+          mma_16816(y[j], yh, dl[2 * j], dl[2 * j + 1]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split_pair(y[e >> 1][(e & 1) * 2], y[e >> 1][(e & 1) * 2 + 1], xh[m][rb][e], xl[m][rb][e]);
+        if (is_v) {
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int col = col0 + (lane >> 2) + (e >> 1) * 8;
+              if (col < dv) p.u0[(unit * CHUNK + rb * 16 + j * 8 + (lane & 3) * 2 + (e & 1)) * dv + col] = y[j][e];
+            }
+        } else {
+          const int at = (rb * 16 + beside + r) * kp + col0 + own;
+          stmatrix_x4_trans(smem_u32(wh + at), xh[m][rb]);
+          stmatrix_x4_trans(smem_u32(wl + at), xl[m][rb]);
+        }
       }
     }
   }
+  __syncthreads();
+  // W and K leave as they lie.
+  const int pieces = 3 * CHUNK * kp / 8;
+  uint4* to = (uint4*)(p.wk + unit * 3 * CHUNK * kp);
+#pragma unroll 4
+  for (int e = tid; e < pieces; e += SOLVE_THREADS) to[e] = ((const uint4*)raw)[e];
 }
 
 // ---------------------------------------------------------------------------------------
@@ -490,10 +614,8 @@ __global__ void __launch_bounds__(SOLVE_THREADS) delta_solve_kernel(const Delta 
 constexpr int PASS_THREADS = 256;
 constexpr size_t SMEM_MOST = 220 * 1024;      // beside a kilobyte of static shared memory
 
-__host__ __device__ inline int pass_channels(int n) { return (n + 31) & ~31; }      // steps of 32 key channels
 __host__ __device__ inline size_t pass_smem(int n, int dvt, int stages) {
-  const int np = pass_channels(n);
-  return 2 * ((size_t)stages * 3 * CHUNK * (np + 8) + (size_t)2 * (np + CHUNK) * (dvt + 8));
+  return 2 * ((size_t)stages * 3 * CHUNK * pitch_of(n) + (size_t)2 * (padded(n) + CHUNK) * (dvt + 8));
 }
 
 // From chunk to chunk, DVT value columns of a head of a request a block. The state lives in the
@@ -509,20 +631,20 @@ __global__ void __launch_bounds__(PASS_THREADS) delta_pass_kernel(const Delta p,
   if (count <= 1) return;
   const int chunks = (count + CHUNK - 1) / CHUNK;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mid = lane >> 3, r = lane & 7;
-  const int n = p.n, dv = p.dv, np = pass_channels(n), kp = np + 8, g = h / (p.heads / p.groups);
+  const int n = p.n, dv = p.dv, np = padded(n), kp = np + 8;
   const size_t stage_size = (size_t)3 * CHUNK * kp;
   __nv_bfloat16* ring = (__nv_bfloat16*)raw;                     // per stage W hi, W lo, K: [CHUNK][kp] each
   __nv_bfloat16* sh = ring + stages * stage_size;                // [np][VP]
   __nv_bfloat16* sl = sh + (size_t)np * VP;
   __nv_bfloat16* uh = sl + (size_t)np * VP;                      // [CHUNK][VP]: exp(c_last - c_j) U_j / |k_j|
   __nv_bfloat16* ul = uh + (size_t)CHUNK * VP;
-  auto fetch = [&](int chunk) {
-    const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h, token0 = (size_t)first + chunk * CHUNK;
-    __nv_bfloat16* to = ring + (stages > 1 ? chunk & 1 : 0) * stage_size;
-    const __nv_bfloat16* w = p.w + unit * 2 * CHUNK * n;
-    fetch_rows(to, kp, w, n, CHUNK, CHUNK, np, n);
-    fetch_rows(to + (size_t)CHUNK * kp, kp, w + (size_t)CHUNK * n, n, CHUNK, CHUNK, np, n);
-    fetch_rows(to + (size_t)2 * CHUNK * kp, kp, (const __nv_bfloat16*)p.k + token0 * p.k_ld + g * n, p.k_ld, CHUNK, count - chunk * CHUNK, np, n);
+  const int pieces = 3 * CHUNK * kp / 8;
+  auto fetch = [&](int chunk) {                                  // W and K of a chunk, as they lie
+    const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
+    const uint32_t to = smem_u32(ring + (stages > 1 ? chunk & 1 : 0) * stage_size) + tid * 16;
+    const uint4* from = (const uint4*)(p.wk + unit * 3 * CHUNK * kp) + tid;
+#pragma unroll 4
+    for (int e = 0; e + tid < pieces; e += PASS_THREADS) cp_async16(to + e * 16, from + e);
     cp_async_commit();
   };
   float* st = p.state + (size_t)p.state_slot[b] * p.slot_stride + (size_t)h * n * dv;
@@ -538,7 +660,8 @@ __global__ void __launch_bounds__(PASS_THREADS) delta_pass_kernel(const Delta p,
         if (row < n && col < dv) x = *(const float2*)(st + (size_t)row * dv + col);
         s[m][j][half * 2] = x.x, s[m][j][half * 2 + 1] = x.y;
       }
-  auto stage_state = [&]() {
+  auto stage_state = [&](int chunk) {    // the state before a chunk: into shared memory, and to the output kernel
+    __nv_bfloat16* out = p.before + ((size_t)chunk_slot(first, i, chunk) * p.heads + h) * 2 * n * dv + d0;
 #pragma unroll
     for (int m = 0; m < 2; ++m) {
       if ((warp + 8 * m) * 16 >= np) break;
@@ -546,51 +669,54 @@ __global__ void __launch_bounds__(PASS_THREADS) delta_pass_kernel(const Delta p,
       for (int j = 0; j < NT; ++j)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          const int at = ((warp + 8 * m) * 16 + (lane >> 2) + half * 8) * VP + j * 8 + (lane & 3) * 2;
+          const int row = (warp + 8 * m) * 16 + (lane >> 2) + half * 8, col = j * 8 + (lane & 3) * 2;
           uint32_t hi, lo;
           split_pair(s[m][j][half * 2], s[m][j][half * 2 + 1], hi, lo);
-          *(uint32_t*)(sh + at) = hi;
-          *(uint32_t*)(sl + at) = lo;
+          *(uint32_t*)(sh + row * VP + col) = hi;
+          *(uint32_t*)(sl + row * VP + col) = lo;
+          if (row < n && d0 + col < dv) {
+            *(uint32_t*)(out + (size_t)row * dv + col) = hi;
+            *(uint32_t*)(out + ((size_t)n + row) * dv + col) = lo;
+          }
         }
     }
   };
-  stage_state();
+  stage_state(0);
   fetch(0);
   const int m0 = (warp & 3) * 16, rows[2] = {m0 + (lane >> 2), m0 + (lane >> 2) + 8};
-  for (int chunk = 0; chunk < chunks; ++chunk) {
+  float2 u0[MINE][2];
+  float last, from[2], inv[2];           // of the chunk: c at its end and at this thread's rows, and 1 / |k|
+  auto ask = [&](int chunk) {            // for what a chunk needs in registers, one chunk ahead
     const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
     const float* vec = p.vec + unit * 2 * CHUNK;
-    float2 u0[MINE][2];
-    float weight[2];
-    const float last = vec[CHUNK - 1];
+    last = vec[CHUNK - 1];
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      weight[half] = exp2f(last - vec[rows[half]]) * vec[CHUNK + rows[half]];
+      from[half] = vec[rows[half]];
+      inv[half] = vec[CHUNK + rows[half]];
 #pragma unroll
       for (int j = 0; j < MINE; ++j) {
         const int col = d0 + ((warp >> 2) + 2 * j) * 8 + (lane & 3) * 2;
         u0[j][half] = col < dv ? *(const float2*)(p.u0 + (unit * CHUNK + rows[half]) * dv + col) : make_float2(0.f, 0.f);
       }
     }
+  };
+  ask(0);
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
+    const float weight[2] = {exp2f(last - from[0]) * inv[0], exp2f(last - from[1]) * inv[1]}, keep = exp2f(last);
     cp_async_wait<0>();
     __syncthreads();                     // this chunk's operands and the state's planes are there; the chunk before is done with
     if (stages > 1 && chunk + 1 < chunks) fetch(chunk + 1);
     const __nv_bfloat16* wh = ring + (stages > 1 ? chunk & 1 : 0) * stage_size;
     const __nv_bfloat16* ks = wh + (size_t)2 * CHUNK * kp;
-    {
-      __nv_bfloat16* out = p.before + unit * 2 * n * dv + d0;
-      for (int e = tid; e < 2 * n * NT; e += PASS_THREADS) {
-        const int plane = e >= n * NT, at = e - plane * n * NT, row = at / NT, c = (at - row * NT) * 8;
-        if (d0 + c < dv) *(uint4*)(out + ((size_t)plane * n + row) * dv + c) = *(const uint4*)((plane ? sl : sh) + row * VP + c);
-      }
-    }
     float acc[MINE][3][4];
 #pragma unroll
     for (int j = 0; j < MINE; ++j)
 #pragma unroll
       for (int x = 0; x < 3; ++x) acc[j][x][0] = acc[j][x][1] = acc[j][x][2] = acc[j][x][3] = 0.f;
     const uint32_t w_at = smem_u32(wh + (size_t)(m0 + (mid & 1) * 8 + r) * kp + (mid >> 1) * 8), w_lo = CHUNK * kp * 2;
-#pragma unroll 2
+#pragma unroll 4
     for (int t = 0; t < np; t += 32) {
       uint32_t ah[2][4], al[2][4];
 #pragma unroll
@@ -630,8 +756,8 @@ __global__ void __launch_bounds__(PASS_THREADS) delta_pass_kernel(const Delta p,
           *(uint32_t*)(out + (size_t)CHUNK * dv) = lo;
         }
       }
+    if (chunk + 1 < chunks) ask(chunk + 1);
     __syncthreads();
-    const float keep = exp2f(last);
 #pragma unroll
     for (int m = 0; m < 2; ++m) {
       const int row0 = (warp + 8 * m) * 16;
@@ -657,7 +783,7 @@ __global__ void __launch_bounds__(PASS_THREADS) delta_pass_kernel(const Delta p,
         }
       }
     }
-    stage_state();                       // its readers are behind the barrier above
+    if (chunk + 1 < chunks) stage_state(chunk + 1);      // its readers are behind the barrier above
     if (stages == 1 && chunk + 1 < chunks) {
       __syncthreads();                   // K is used up
       fetch(chunk + 1);
@@ -779,7 +905,7 @@ __global__ void __launch_bounds__(OUT_THREADS) delta_output_kernel(const Delta p
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int token = t * 16 + w * 8 + (lane & 3) * 2 + (e & 1), half = e >> 1;
-        s[w][e] = token <= rows[half] ? s[w][e] * (scale[half] * k_inv[token] * exp2f(at_row[half] - cumulative[token])) : 0.f;
+        s[w][e] = token <= rows[half] ? s[w][e] * (scale[half] * k_inv[token] * fast_exp2(at_row[half] - cumulative[token])) : 0.f;
       }
     uint32_t hi[4], lo[4];
 #pragma unroll
@@ -878,31 +1004,32 @@ PAE_EXPORT int pae_gated_delta_step(float* o, float* state, long long slot_strid
 
 // 1 when the chunked kernels take these sizes: rows of 16-byte pieces, up to 256 key channels.
 PAE_EXPORT int pae_gated_delta_chunked_supports(int n, int dv, int q_ld, int k_ld, int v_ld, long long slot_stride) {
-  return n % 8 == 0 && dv % 8 == 0 && n <= 256 && q_ld % 8 == 0 && k_ld % 8 == 0 && v_ld % 8 == 0 && slot_stride % 2 == 0 ? 1 : 0;
+  return n % 8 == 0 && dv % 8 == 0 && n <= 256 && solve_smem(n, dv) <= SMEM_MOST && q_ld % 8 == 0 && k_ld % 8 == 0 && v_ld % 8 == 0 && slot_stride % 2 == 0 ? 1 : 0;
 }
 
 PAE_EXPORT int pae_gated_delta_chunk() { return CHUNK; }
+PAE_EXPORT int pae_gated_delta_pitch(int n) { return pitch_of(n); }
 
 // The entries that bring more than one token, bfloat16. list: `listed` entries to look at (null: all, and
-// those of one token are passed over). Scratch for tokens / 64 + listed chunks, per chunk and head: w bfloat16
-// [2, 64, n], u0 floats [64, dv], u bfloat16 [2, 64, dv], before bfloat16 [2, n, dv], vec floats [2, 64]. Three launches.
+// those of one token are passed over). Scratch for tokens / 64 + listed chunks, per chunk and head: wk bfloat16
+// [3, 64, pitch], u0 floats [64, dv], u bfloat16 [2, 64, dv], before bfloat16 [2, n, dv], vec floats [2, 64]. Three launches.
 PAE_EXPORT int pae_gated_delta_chunked(float* o, float* state, long long slot_stride, const void* q, int q_ld, const void* k, int k_ld,
                                        const void* v, int v_ld, const float* log_decay, const float* beta, float key_eps, float q_scale,
                                        const int* q_start, const int* state_slot, const int* list, int listed, int max_q_len, int heads,
-                                       int groups, int n, int dv, void* w, float* u0, void* u, void* before, float* vec, void* stream) {
+                                       int groups, int n, int dv, void* wk, float* u0, void* u, void* before, float* vec, void* stream) {
   if (listed == 0 || max_q_len <= 1) return 0;
   Delta p = delta_of(o, state, slot_stride, q, q_ld, k, k_ld, v, v_ld, log_decay, beta, key_eps, q_scale, q_start, state_slot, heads, groups, n, dv);
   p.list = list;
-  p.w = (__nv_bfloat16*)w, p.u0 = u0, p.u = (__nv_bfloat16*)u, p.before = (__nv_bfloat16*)before, p.vec = vec;
+  p.wk = (__nv_bfloat16*)wk, p.u0 = u0, p.u = (__nv_bfloat16*)u, p.before = (__nv_bfloat16*)before, p.vec = vec;
   if (int err = check_delta(p, listed)) return err;
   if (!pae_gated_delta_chunked_supports(n, dv, q_ld, k_ld, v_ld, slot_stride))
     return fail(2, "gated_delta_chunked: heads of %d key and %d value channels", n, dv);
-  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)state | (uintptr_t)w | (uintptr_t)u0 | (uintptr_t)u | (uintptr_t)before) & 15)
+  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)state | (uintptr_t)wk | (uintptr_t)u0 | (uintptr_t)u | (uintptr_t)before) & 15)
     return fail(2, "gated_delta_chunked: an operand does not start on a 16-byte boundary");
   cudaStream_t s = (cudaStream_t)stream;
-  const int chunks = (max_q_len + CHUNK - 1) / CHUNK, np = (n + 15) & ~15;
-  if (int err = allow_smem(delta_solve_kernel, solve_smem(256), "gated_delta_chunked")) return err;
-  launch_kernel(delta_solve_kernel, dim3(chunks, heads, listed), SOLVE_THREADS, solve_smem(np), s, p);
+  const int chunks = (max_q_len + CHUNK - 1) / CHUNK;
+  if (int err = allow_smem(delta_solve_kernel, SMEM_MOST, "gated_delta_chunked")) return err;
+  launch_kernel(delta_solve_kernel, dim3(chunks, heads, listed), SOLVE_THREADS, solve_smem(n, dv), s, p);
   if (int err = check_launch("gated_delta_solve")) return err;
   // wider blocks read W and K fewer times; narrow ones keep the SMs busy while the heads are few
   const bool wide = (long long)listed * heads * ((dv + 31) / 32) >= 148;

@@ -8,10 +8,11 @@
 //
 // with rms(v) = v / sqrt(mean(v^2) + eps). A branch may be the planes of a split product, which are added
 // in their order first. Every piece is optional, and a launch with the pieces that a caller has is what
-// runs: the sum of branches alone, the residual alone, the rounding alone. A block owns a row and keeps it
-// in shared memory between the passes; a thread only ever touches its own columns there, so the barriers
-// are the ones inside the sums. The stream and all arithmetic are float32 (sums of squares double),
-// every read is rounded once.
+// runs: the sum of branches alone, the residual alone, the rounding alone. A block owns a row. Rows of up
+// to 8,192 columns that split into aligned 16-byte pieces, with one or two branches, stay in registers,
+// all of their loads asked for before the first sum; any other row stays in shared memory between the
+// passes, where a thread only ever touches its own columns. The stream and all arithmetic are float32 (sums
+// of squares double), every read is rounded once.
 #include "common.cuh"
 
 using namespace pae;
@@ -48,6 +49,9 @@ __device__ __forceinline__ double row_sum(double v, double* scratch) {
   for (int i = 0; i < warps; ++i) total += scratch[i];     // every thread adds in the same order
   return total;
 }
+
+// Rounded step by step, so that every form of the kernel gives the same bits.
+__device__ __forceinline__ float normed(float v, float inv, float w) { return __fmul_rn(__fmul_rn(v, inv), w); }
 
 template <int VEC>
 struct Piece {
@@ -108,7 +112,8 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNorm p) {
   __shared__ double scratch[32];
   const int width = p.width, step = blockDim.x * VEC, c0 = threadIdx.x * VEC;
   const size_t at = (size_t)blockIdx.x * width;
-  auto inverse = [&](double squares, float eps) { return (float)(1.0 / sqrt(row_sum(squares, scratch) / (double)width + (double)eps)); };
+  const double part = 1.0 / (double)width;
+  auto inverse = [&](double squares, float eps) { return 1.f / sqrtf((float)fma(row_sum(squares, scratch), part, (double)eps)); };
   float inv[MAX_BRANCHES];
   for (int b = 0; b < p.branches; ++b) {
     double squares = 0.0;
@@ -134,10 +139,10 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNorm p) {
         if (p.w[b] != nullptr) {
           const Piece<VEC> w = get<VEC>(p.w[b] + c);
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) v.v[e] += p.scale[b] * (s.v[e] * inv[b] * w.v[e]);
+          for (int e = 0; e < VEC; ++e) v.v[e] = fmaf(p.scale[b], normed(s.v[e], inv[b], w.v[e]), v.v[e]);
         } else {
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) v.v[e] += p.scale[b] * s.v[e];
+          for (int e = 0; e < VEC; ++e) v.v[e] = fmaf(p.scale[b], s.v[e], v.v[e]);
         }
       }
 #pragma unroll
@@ -161,10 +166,10 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNorm p) {
       if (p.post_w != nullptr) {
         const Piece<VEC> w = get<VEC>(p.post_w + c);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) x.v[e] += p.mult * (v.v[e] * post * w.v[e]);
+        for (int e = 0; e < VEC; ++e) x.v[e] = fmaf(p.mult, normed(v.v[e], post, w.v[e]), x.v[e]);
       } else {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) x.v[e] += p.mult * v.v[e];
+        for (int e = 0; e < VEC; ++e) x.v[e] = fmaf(p.mult, v.v[e], x.v[e]);
       }
     }
     if (p.x_new != nullptr) put<VEC>(p.x_new + at + c, x);
@@ -183,9 +188,164 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNorm p) {
     Piece<VEC> x = get<VEC>(row + c);
     const Piece<VEC> w = get<VEC>(p.read_w + c);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) x.v[e] = x.v[e] * last * w.v[e];
+    for (int e = 0; e < VEC; ++e) x.v[e] = normed(x.v[e], last, w.v[e]);
     put<VEC>(read + c, x);
   }
+}
+
+// The row in registers: PER pieces of four columns a thread, BRANCHES outputs.
+template <typename TO, int PER, int BRANCHES>
+__global__ void __launch_bounds__(PER <= 4 ? 512 : 256) post_norm_row_kernel(const PostNorm p) {
+  dependent_launch_prologue();
+  constexpr int AHEAD = PER == 1 ? 8 : (PER == 2 ? 4 : 1);      // planes asked for at a time (few rows have planes, and few pieces a thread)
+  __shared__ double scratch[3][BRANCHES][16];      // a set per sum: one barrier each
+  const int width = p.width, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const size_t at = (size_t)blockIdx.x * width;
+  const int c0 = threadIdx.x * 4, step = blockDim.x * 4;
+  const double part = 1.0 / (double)width;
+  auto inverse = [&](double total, float eps) { return 1.f / sqrtf((float)fma(total, part, (double)eps)); };
+  Piece<4> y[BRANCHES][PER], x[PER];
+#pragma unroll
+  for (int b = 0; b < BRANCHES; ++b)
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (c0 + i * step < width) y[b][i] = get<4>(p.y[b] + at + c0 + i * step);
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    x[i].v[0] = x[i].v[1] = x[i].v[2] = x[i].v[3] = 0.f;
+    if (p.x != nullptr && c0 + i * step < width) x[i] = get<4>(p.x + at + c0 + i * step);
+  }
+  double squares[BRANCHES];
+#pragma unroll
+  for (int b = 0; b < BRANCHES; ++b) {
+    const float* from = p.y[b] + at + c0;
+    for (int k = 1; k < p.planes[b]; k += AHEAD) {      // the planes in their order
+      Piece<4> more[AHEAD][PER];
+#pragma unroll
+      for (int j = 0; j < AHEAD; ++j)
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+          if (k + j < p.planes[b] && c0 + i * step < width) more[j][i] = get<4>(from + (size_t)(k + j) * p.total + i * step);
+#pragma unroll
+      for (int j = 0; j < AHEAD; ++j)
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+          if (k + j < p.planes[b] && c0 + i * step < width)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[b][i].v[e] += more[j][i].v[e];
+    }
+    squares[b] = 0.0;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (c0 + i * step < width)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) squares[b] = fma((double)y[b][i].v[e], (double)y[b][i].v[e], squares[b]);
+  }
+  auto share = [&](double v, int set, int b) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    if (lane == 0) scratch[set][b][warp] = v;
+  };
+  auto total = [&](int set, int b) {
+    double sum = 0.0;
+    for (int w = 0; w < warps; ++w) sum += scratch[set][b][w];      // every thread adds in the same order
+    return sum;
+  };
+  const bool own_norms = p.w[0] != nullptr || (BRANCHES > 1 && p.w[BRANCHES - 1] != nullptr);      // some branch has a norm of its own
+  const bool plain = BRANCHES == 1 && !own_norms && p.scale[0] == 1.f;
+  if (own_norms || (plain && p.post_w != nullptr)) {
+#pragma unroll
+    for (int b = 0; b < BRANCHES; ++b) share(squares[b], 0, b);
+    __syncthreads();
+  }
+  float post = 0.f;
+  if (plain) {
+    if (p.post_w != nullptr) post = inverse(total(0, 0), p.post_eps);
+  } else {
+    double sum = 0.0;
+    float inv[BRANCHES];
+#pragma unroll
+    for (int b = 0; b < BRANCHES; ++b) inv[b] = p.w[b] != nullptr ? inverse(total(0, b), p.branch_eps) : 1.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      if (c0 + i * step >= width) break;
+      Piece<4> v;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v.v[e] = 0.f;
+#pragma unroll
+      for (int b = 0; b < BRANCHES; ++b) {
+        if (p.w[b] != nullptr) {
+          const Piece<4> w = get<4>(p.w[b] + c0 + i * step);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v.v[e] = fmaf(p.scale[b], normed(y[b][i].v[e], inv[b], w.v[e]), v.v[e]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v.v[e] = fmaf(p.scale[b], y[b][i].v[e], v.v[e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sum = fma((double)v.v[e], (double)v.v[e], sum);
+      y[0][i] = v;
+    }
+    if (p.post_w != nullptr) {
+      share(sum, 1, 0);
+      __syncthreads();
+      post = inverse(total(1, 0), p.post_eps);
+    }
+  }
+  double sum = 0.0;
+  TO* read = (TO*)p.read + at;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = c0 + i * step;
+    if (c >= width) break;
+    if (p.post_w != nullptr) {
+      const Piece<4> w = get<4>(p.post_w + c);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[i].v[e] = fmaf(p.mult, normed(y[0][i].v[e], post, w.v[e]), x[i].v[e]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[i].v[e] = fmaf(p.mult, y[0][i].v[e], x[i].v[e]);
+    }
+    if (p.x_new != nullptr) put<4>(p.x_new + at + c, x[i]);
+    if (p.read == nullptr) continue;
+    if (p.read_w == nullptr) {
+      put<4>(read + c, x[i]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sum = fma((double)x[i].v[e], (double)x[i].v[e], sum);
+    }
+  }
+  if (p.read == nullptr || p.read_w == nullptr) return;
+  share(sum, 2, 0);
+  __syncthreads();
+  const float last = inverse(total(2, 0), p.read_eps);
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = c0 + i * step;
+    if (c >= width) break;
+    const Piece<4> w = get<4>(p.read_w + c);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[i].v[e] = normed(x[i].v[e], last, w.v[e]);
+    put<4>(read + c, x[i]);
+  }
+}
+
+template <typename TO, int BRANCHES>
+int launch_row(const PostNorm& p, int rows, cudaStream_t s) {
+  const int pieces = p.width / 4;
+  // many rows: a few warps a row, so that an SM holds many; few rows: as many threads as there are pieces
+  const int threads = rows > 64 ? (pieces <= 1024 ? 128 : 256) : (pieces <= 128 ? 128 : pieces <= 256 ? 256 : 512);
+  switch ((pieces + threads - 1) / threads) {
+    case 1: launch_kernel(post_norm_row_kernel<TO, 1, BRANCHES>, rows, threads, 0, s, p); break;
+    case 2: launch_kernel(post_norm_row_kernel<TO, 2, BRANCHES>, rows, threads, 0, s, p); break;
+    case 3: launch_kernel(post_norm_row_kernel<TO, 3, BRANCHES>, rows, threads, 0, s, p); break;
+    case 4: launch_kernel(post_norm_row_kernel<TO, 4, BRANCHES>, rows, threads, 0, s, p); break;
+    case 5:
+    case 6: launch_kernel(post_norm_row_kernel<TO, 6, BRANCHES>, rows, threads, 0, s, p); break;
+    default: launch_kernel(post_norm_row_kernel<TO, 8, BRANCHES>, rows, threads, 0, s, p); break;
+  }
+  return check_launch("post_norm");
 }
 
 constexpr size_t SMEM_MOST = 200 * 1024;
@@ -223,6 +383,11 @@ PAE_EXPORT int pae_post_norm(float* x_new, void* read, const float* x, int branc
   for (int b = 0; b < MAX_BRANCHES; ++b) {
     if (b < branches && (p.y[b] == nullptr || p.planes[b] < 1)) return fail(2, "post_norm: branch %d has %d planes", b, p.planes[b]);
     wide = wide && aligned16(p.y[b]) && aligned16(p.w[b]);
+  }
+  if (wide && width <= 8192 && (branches == 1 || branches == 2)) {
+    cudaStream_t s = (cudaStream_t)stream;
+    if (read_dtype == kF32) return branches == 1 ? launch_row<float, 1>(p, rows, s) : launch_row<float, 2>(p, rows, s);
+    return branches == 1 ? launch_row<__nv_bfloat16, 1>(p, rows, s) : launch_row<__nv_bfloat16, 2>(p, rows, s);
   }
   const size_t bytes = sizeof(float) * (size_t)(branches > 1 ? branches : 1) * width;
   if (bytes > SMEM_MOST) return fail(2, "post_norm: %d rows of %d do not fit shared memory", branches, width);

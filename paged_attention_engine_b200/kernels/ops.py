@@ -1703,12 +1703,12 @@ def gated_delta(q, k, v, log_decay, beta, state, q_start, state_slot, num_seqs: 
         listed = multi_index.numel()
     chunk = lib.pae_gated_delta_chunk()
     units = (tokens // chunk + listed) * num_heads
-    w = torch.empty(units * 2 * chunk * key_dim, dtype=torch.bfloat16, device=o.device)
+    wk = torch.empty(units * 3 * chunk * lib.pae_gated_delta_pitch(key_dim), dtype=torch.bfloat16, device=o.device)
     u0 = torch.empty(units * chunk * value_dim, dtype=torch.float32, device=o.device)
     u = torch.empty(units * 2 * chunk * value_dim, dtype=torch.bfloat16, device=o.device)
     before = torch.empty(units * 2 * key_dim * value_dim, dtype=torch.bfloat16, device=o.device)
     vec = torch.empty(units * 2 * chunk, dtype=torch.float32, device=o.device)
-    _check(lib, lib.pae_gated_delta_chunked(*what, _ptr(multi_index), listed, max_q_len, *sizes, _ptr(w), _ptr(u0), _ptr(u), _ptr(before),
+    _check(lib, lib.pae_gated_delta_chunked(*what, _ptr(multi_index), listed, max_q_len, *sizes, _ptr(wk), _ptr(u0), _ptr(u), _ptr(before),
                                             _ptr(vec), _stream()), 3)
     return o
 
