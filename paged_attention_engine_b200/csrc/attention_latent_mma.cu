@@ -56,6 +56,8 @@ struct LatentParams {
   float* part_sum;
 };
 
+// WINDOWED is known when compiled: the window's comparisons cost a causal prompt a fifth of its time.
+template <bool WINDOWED>
 __global__ void __launch_bounds__(THREADS) latent_kernel(const LatentParams p) {
   dependent_launch_prologue();
   extern __shared__ __align__(128) uint8_t smem[];
@@ -70,7 +72,7 @@ __global__ void __launch_bounds__(THREADS) latent_kernel(const LatentParams p) {
   const int rows = single ? min(ROWS, p.heads - head0) : min(ROWS, q_count - tile * ROWS);
   const int pos0 = p.q_pos0[b] + tile * ROWS;
   const int kv_end = single ? min(p.kv_len[b], pos0 + 1) : min(p.kv_len[b], pos0 + rows);
-  const int kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;      // the first key that the block's first row sees
+  const int kv_begin = WINDOWED ? max(0, pos0 - p.window + 1) : 0;      // the first key that the block's first row sees
   const int D = p.D, DV = p.DV;
   const int chunks = D >> 3;                                           // 16-byte chunks of a row
   const int row_bytes = D * 2 + 16;
@@ -96,7 +98,7 @@ __global__ void __launch_bounds__(THREADS) latent_kernel(const LatentParams p) {
   auto fetch = [&](int stage, int key0) {
     const int key = key0 + f_row;
     uint8_t* dst = k_stage + (size_t)stage * TILE * row_bytes + f_row * row_bytes;
-    if (key < kv_end && key >= kv_begin) {
+    if (key < kv_end && (!WINDOWED || key >= kv_begin)) {
       const int index = key / p.page_size;
       const int page = checked_page(table[checked_table_index(index, p.table_width)]);
       const __nv_bfloat16* src = p.keys + ((size_t)page * p.page_size + (key - index * p.page_size)) * D;
@@ -118,6 +120,7 @@ __global__ void __launch_bounds__(THREADS) latent_kernel(const LatentParams p) {
   const int row0 = group * GROUP_ROWS;                                 // this group's first row of the block
   const bool working = row0 < rows;                                    // a group without rows only helps to fetch
   const int my_pos[2] = {single ? pos0 : pos0 + row0 + (lane >> 2), single ? pos0 : pos0 + row0 + (lane >> 2) + 8};
+  const int first_pos = single ? pos0 : pos0 + row0;
   const int last_pos = single ? pos0 : pos0 + min(rows, row0 + GROUP_ROWS) - 1;
   const int c2 = (lane & 3) * 2;
   const int mid = lane >> 3, r8 = lane & 7;
@@ -181,15 +184,27 @@ __global__ void __launch_bounds__(THREADS) latent_kernel(const LatentParams p) {
         s[1][0] = hi.x, s[1][1] = hi.y, s[1][2] = hi.z, s[1][3] = hi.w;
       }
       float block_max[2] = {-FLT_MAX, -FLT_MAX};
+      // every row of the group sees all 16 keys: nothing to compare
+      const bool open = key0 + 15 <= first_pos && key0 + 16 <= kv_end && (!WINDOWED || key0 + p.window > last_pos);
+      if (open) {
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
+        for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const int half = j >> 1, key = key0 + i * 8 + c2 + (j & 1);
-          const bool seen = key < kv_end && key <= my_pos[half] && (p.window <= 0 || key + p.window > my_pos[half]);
-          s[i][j] = seen ? s[i][j] * scale2 : -FLT_MAX;
-          block_max[half] = fmaxf(block_max[half], s[i][j]);
-        }
+          for (int j = 0; j < 4; ++j) {
+            s[i][j] *= scale2;
+            block_max[j >> 1] = fmaxf(block_max[j >> 1], s[i][j]);
+          }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int half = j >> 1, key = key0 + i * 8 + c2 + (j & 1);
+            const bool seen = key < kv_end && key <= my_pos[half] && (!WINDOWED || key + p.window > my_pos[half]);
+            s[i][j] = seen ? s[i][j] * scale2 : -FLT_MAX;
+            block_max[half] = fmaxf(block_max[half], s[i][j]);
+          }
+      }
       float rescale[2];
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
@@ -205,7 +220,7 @@ __global__ void __launch_bounds__(THREADS) latent_kernel(const LatentParams p) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int half = j >> 1;
-          const float e = s[i][j] == -FLT_MAX ? 0.f : fast_exp2(s[i][j] - row_max[half]);
+          const float e = !open && s[i][j] == -FLT_MAX ? 0.f : fast_exp2(s[i][j] - row_max[half]);
           s[i][j] = e;
           block_sum[half] += e;
         }
@@ -342,11 +357,13 @@ PAE_EXPORT int pae_paged_attention_latent_mma(void* out, const void* q, const vo
     p.part_sum = p.part_max + units;
   }
   const size_t bytes = smem_bytes(d);
-  if (int err = allow_smem(latent_kernel, 200 * 1024, "paged_attention_latent_mma")) return err;
+  if (int err = allow_smem(latent_kernel<false>, 200 * 1024, "paged_attention_latent_mma")) return err;
+  if (int err = allow_smem(latent_kernel<true>, 200 * 1024, "paged_attention_latent_mma")) return err;
   cudaStream_t s = (cudaStream_t)stream;
   const int q_tiles = (max_q_len + ROWS - 1) / ROWS;
   dim3 grid(scratch != nullptr ? max(q_tiles, splits) : q_tiles, heads, seqs);
-  launch_kernel(latent_kernel, grid, THREADS, bytes, s, p);
+  if (p.window > 0) launch_kernel(latent_kernel<true>, grid, THREADS, bytes, s, p);
+  else launch_kernel(latent_kernel<false>, grid, THREADS, bytes, s, p);
   if (int err = check_launch("paged_attention_latent_mma")) return err;
   if (scratch != nullptr) {
     const int threads = dv >= 512 ? 512 : (dv + 31) / 32 * 32;       // a column a thread

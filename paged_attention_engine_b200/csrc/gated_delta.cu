@@ -58,9 +58,9 @@ struct Delta {
   float key_eps, q_scale;
   // chunked, per (chunk slot, head)
   __nv_bfloat16* wk;         // [3, 64, pitch]: W as a sum of two, and K
-  float* u0;                 // [64, dv]
-  __nv_bfloat16* u;          // [2, 64, dv]: U as a sum of two
-  __nv_bfloat16* before;     // [2, n, dv]: the state before the chunk, as a sum of two
+  float* u0;                 // [dv, 64]
+  __nv_bfloat16* u;          // [2, dv, 64]: U as a sum of two
+  __nv_bfloat16* before;     // [2, dv, n]: the state before the chunk, as a sum of two
   float* vec;                // [2, 64]: c in units of log 2, and 1 / |k|
 };
 
@@ -369,6 +369,22 @@ __device__ __forceinline__ void fetch_rows(__nv_bfloat16* to, int pitch, const _
   }
 }
 
+// The squared length of row t of a chunk's keys or queries in shared memory, by four neighbouring threads.
+__device__ __forceinline__ float row_squares(const __nv_bfloat16* rows, int pitch, int cols, int t) {
+  float sum = 0.f;
+  for (int e = (threadIdx.x & 3) * 8; e < cols; e += 32) {
+    const uint4 eight = *(const uint4*)(rows + t * pitch + e);
+    const __nv_bfloat162* two = (const __nv_bfloat162*)&eight;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = __bfloat1622float2(two[j]);
+      sum = fmaf(f.x, f.x, fmaf(f.y, f.y, sum));
+    }
+  }
+  sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+  return sum + __shfl_xor_sync(0xffffffffu, sum, 2);
+}
+
 // Key channels of a chunk's operands in scratch and in the kernels that share them: steps of 32, and a row's
 // pitch, padded so that the eight rows of an ldmatrix fall into different banks.
 __host__ __device__ inline int padded(int n) { return (n + 31) & ~31; }
@@ -437,20 +453,9 @@ __global__ void __launch_bounds__(SOLVE_THREADS, 2) delta_solve_kernel(const Del
   }
   cp_async_wait<1>();
   __syncthreads();
-  {  // lengths: four threads a token
+  {
     const int t = tid >> 2;
-    float kk = 0.f;
-    for (int e = (tid & 3) * 8; e < np; e += 32) {
-      const uint4 eight = *(const uint4*)(ks + t * kp + e);
-      const __nv_bfloat162* two = (const __nv_bfloat162*)&eight;
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float2 f = __bfloat1622float2(two[j]);
-        kk = fmaf(f.x, f.x, fmaf(f.y, f.y, kk));
-      }
-    }
-    kk += __shfl_xor_sync(0xffffffffu, kk, 1);
-    kk += __shfl_xor_sync(0xffffffffu, kk, 2);
+    const float kk = row_squares(ks, kp, np, t);
     if ((tid & 3) == 0) {
       const float inv = inverse_root(kk + p.key_eps);
       k_inv[t] = inv;
@@ -538,14 +543,14 @@ __global__ void __launch_bounds__(SOLVE_THREADS, 2) delta_solve_kernel(const Del
         const int at = (rb * 16 + beside + r) * L_PITCH + c * 16 + own;
         ldmatrix_x4(bh, smem_u32(ah + at));
         ldmatrix_x4(bl, smem_u32(al + at));
+        // the three products of a sum stand four others apart
 #pragma unroll
-        for (int m = 0; m < 2; ++m)
+        for (int x = 0; x < 3; ++x)
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            mma_16816(sum[m][j], xh[m][c], bh[2 * j], bh[2 * j + 1]);
-            mma_16816(sum[m][j], xl[m][c], bh[2 * j], bh[2 * j + 1]);
-            mma_16816(sum[m][j], xh[m][c], bl[2 * j], bl[2 * j + 1]);
-          }
+          for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+              mma_16816(sum[m][j], x == 1 ? xl[m][c] : xh[m][c], x == 2 ? bl[2 * j] : bh[2 * j], x == 2 ? bl[2 * j + 1] : bh[2 * j + 1]);
       }
       uint32_t dh[4], dl[4];
       {
@@ -577,21 +582,21 @@ __global__ void __launch_bounds__(SOLVE_THREADS, 2) delta_solve_kernel(const Del
 #pragma unroll
         for (int e = 0; e < 4; ++e) split_pair(y[e >> 1][(e & 1) * 2], y[e >> 1][(e & 1) * 2 + 1], yh[e], yl[e]);
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          mma_16816(y[j], yh, dh[2 * j], dh[2 * j + 1]);
-          mma_16816(y[j], yl, dh[2 * j], dh[2 * j + 1]);
-          mma_16816(y[j], yh, dl[2 * j], dl[2 * j + 1]);
-        }
+        for (int x = 0; x < 3; ++x)
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+            mma_16816(y[j], x == 1 ? yl : yh, x == 2 ? dl[2 * j] : dh[2 * j], x == 2 ? dl[2 * j + 1] : dh[2 * j + 1]);
 #pragma unroll
         for (int e = 0; e < 4; ++e) split_pair(y[e >> 1][(e & 1) * 2], y[e >> 1][(e & 1) * 2 + 1], xh[m][rb][e], xl[m][rb][e]);
         if (is_v) {
 #pragma unroll
-          for (int j = 0; j < 2; ++j)
+          for (int half = 0; half < 2; ++half) {
+            const int col = col0 + (lane >> 2) + half * 8;
+            if (col >= dv) continue;
+            float* to = p.u0 + (unit * dv + col) * CHUNK + rb * 16 + (lane & 3) * 2;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              const int col = col0 + (lane >> 2) + (e >> 1) * 8;
-              if (col < dv) p.u0[(unit * CHUNK + rb * 16 + j * 8 + (lane & 3) * 2 + (e & 1)) * dv + col] = y[j][e];
-            }
+            for (int j = 0; j < 2; ++j) *(float2*)(to + j * 8) = make_float2(y[j][half * 2], y[j][half * 2 + 1]);
+          }
         } else {
           const int at = (rb * 16 + beside + r) * kp + col0 + own;
           stmatrix_x4_trans(smem_u32(wh + at), xh[m][rb]);
@@ -611,179 +616,185 @@ __global__ void __launch_bounds__(SOLVE_THREADS, 2) delta_solve_kernel(const Del
 // ---------------------------------------------------------------------------------------
 // chunked: pass
 // ---------------------------------------------------------------------------------------
-constexpr int PASS_THREADS = 256;
-constexpr size_t SMEM_MOST = 220 * 1024;      // beside a kilobyte of static shared memory
+constexpr int PASS_THREADS = 256, PASS_WARPS = PASS_THREADS / 32;
+constexpr int PASS_COLUMNS = 16;              // value columns of a block
+constexpr int PART_PITCH = CHUNK + 8;         // floats between rows of a partial product
+constexpr int U_PITCH = CHUNK + 8;
+constexpr size_t SMEM_MOST = 220 * 1024;      // beside some kilobytes of static shared memory
 
-__host__ __device__ inline size_t pass_smem(int n, int dvt, int stages) {
-  return 2 * ((size_t)stages * 3 * CHUNK * pitch_of(n) + (size_t)2 * (padded(n) + CHUNK) * (dvt + 8));
+__host__ __device__ inline size_t pass_smem(int n, int stages) {
+  return 2 * (size_t)stages * 3 * CHUNK * pitch_of(n) + sizeof(float) * (size_t)PASS_WARPS * PASS_COLUMNS * PART_PITCH;
 }
 
-// From chunk to chunk, DVT value columns of a head of a request a block. The state lives in the
-// accumulators of its update (a warp 16 or 32 key channels of it); a copy as two bfloat16 planes in
-// shared memory is the operand of W S, and goes to the output kernel from there.
-template <int DVT>
-__global__ void __launch_bounds__(PASS_THREADS) delta_pass_kernel(const Delta p, int stages) {
+// From chunk to chunk, 16 value columns of a head of a request a block. The state never leaves the registers: a
+// warp holds S^T, 16 columns by its own 16 key channels (or twice as many), as the accumulators of the update S^T <-
+// exp(c_last) S^T + U^T K, which as they lie are the operand of its share of (W S)^T = S^T W^T. The warps' shares
+// are added up through shared memory.
+__global__ void __launch_bounds__(PASS_THREADS, 2) delta_pass_kernel(const Delta p, int stages) {
   dependent_launch_prologue();
   extern __shared__ __align__(16) unsigned char raw[];
-  constexpr int VP = DVT + 8, NT = DVT / 8, MINE = DVT / 16;      // MINE: 8-column tiles of W S that a warp computes
-  const int d0 = blockIdx.x * DVT, h = blockIdx.y, i = blockIdx.z, b = p.list != nullptr ? p.list[i] : i;
+  __shared__ __align__(16) __nv_bfloat16 us[2][PASS_COLUMNS][U_PITCH];      // exp(c_last - c_j) U_j / |k_j| as a sum of two
+  __shared__ __align__(16) float weight[CHUNK];                             // exp(c_last - c_j) / |k_j|
+  const int d0 = blockIdx.x * PASS_COLUMNS, h = blockIdx.y, i = blockIdx.z, b = p.list != nullptr ? p.list[i] : i;
   const int first = p.q_start[b], count = p.q_start[b + 1] - first;
   if (count <= 1) return;
   const int chunks = (count + CHUNK - 1) / CHUNK;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mid = lane >> 3, r = lane & 7;
-  const int n = p.n, dv = p.dv, np = padded(n), kp = np + 8;
+  const int n = p.n, dv = p.dv, np = padded(n), kp = np + 8, tiles = np / 16;
   const size_t stage_size = (size_t)3 * CHUNK * kp;
   __nv_bfloat16* ring = (__nv_bfloat16*)raw;                     // per stage W hi, W lo, K: [CHUNK][kp] each
-  __nv_bfloat16* sh = ring + stages * stage_size;                // [np][VP]
-  __nv_bfloat16* sl = sh + (size_t)np * VP;
-  __nv_bfloat16* uh = sl + (size_t)np * VP;                      // [CHUNK][VP]: exp(c_last - c_j) U_j / |k_j|
-  __nv_bfloat16* ul = uh + (size_t)CHUNK * VP;
-  const int pieces = 3 * CHUNK * kp / 8;
-  auto fetch = [&](int chunk) {                                  // W and K of a chunk, as they lie
-    const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
-    const uint32_t to = smem_u32(ring + (stages > 1 ? chunk & 1 : 0) * stage_size) + tid * 16;
-    const uint4* from = (const uint4*)(p.wk + unit * 3 * CHUNK * kp) + tid;
+  float* part = (float*)(ring + stages * stage_size);            // [PASS_WARPS][PASS_COLUMNS][PART_PITCH]
+  const int parts = min(tiles, PASS_WARPS);
+  // A thread adds up, and turns into U, four tokens of one column.
+  const int my_col = tid >> 4, my_row = (tid & 15) * 4;
+  const bool my_valid = d0 + my_col < dv;
+  // What lies in scratch per chunk and head: a chunk on, `heads` units on.
+  const size_t unit0 = (size_t)chunk_slot(first, i, 0) * p.heads + h, heads = p.heads;
+  const int pieces = 3 * CHUNK * kp / 8, whole = pieces / PASS_THREADS * PASS_THREADS;
+  const uint4* wk_at = (const uint4*)(p.wk + unit0 * 3 * CHUNK * kp) + tid;
+  const float* vec_at = p.vec + unit0 * 2 * CHUNK;
+  const float* u0_at = p.u0 + (unit0 * dv + d0 + my_col) * CHUNK + my_row;
+  __nv_bfloat16* u_at = p.u + (unit0 * 2 * dv + d0 + my_col) * CHUNK + my_row;
+  __nv_bfloat16* before_at = p.before + (unit0 * 2 * dv + d0 + (lane >> 2)) * n + warp * 16 + (lane & 3) * 2;
+  const size_t wk_step = heads * pieces, vec_step = heads * 2 * CHUNK, u0_step = heads * dv * CHUNK, u_step = 2 * u0_step, before_step = heads * 2 * dv * n;
+  const size_t lo_state = (size_t)dv * n, lo_u = (size_t)dv * CHUNK;
+  const uint32_t ring_at = smem_u32(ring) + tid * 16, ring_other = stages > 1 ? (uint32_t)(stage_size * 2) : 0;
+  auto fetch = [&](int chunk) {                                  // W and K of the next chunk, as they lie
+    const uint32_t to = ring_at + (chunk & 1 ? ring_other : 0);
 #pragma unroll 4
-    for (int e = 0; e + tid < pieces; e += PASS_THREADS) cp_async16(to + e * 16, from + e);
+    for (int e = 0; e < whole; e += PASS_THREADS) cp_async16(to + e * 16, wk_at + e);
+    if (whole + tid < pieces) cp_async16(to + whole * 16, wk_at + whole);
     cp_async_commit();
+    wk_at += wk_step;
+  };
+  // What a chunk needs in registers, asked for a chunk ahead: U0, c at its end and at token tid, and 1 / |k| there.
+  float4 u0 = make_float4(0.f, 0.f, 0.f, 0.f), next_u0 = u0;
+  float next_last = 0.f, next_c = 0.f, next_inv = 0.f;
+  auto ask = [&]() {
+    next_last = vec_at[CHUNK - 1];
+    next_c = vec_at[tid & (CHUNK - 1)];
+    next_inv = vec_at[CHUNK + (tid & (CHUNK - 1))];
+    if (my_valid) next_u0 = *(const float4*)u0_at;
+    vec_at += vec_step;
+    u0_at += u0_step;
   };
   float* st = p.state + (size_t)p.state_slot[b] * p.slot_stride + (size_t)h * n * dv;
-  float s[2][NT][4];
+  // s[m][j][e]: column (lane >> 2) + (e >> 1) 8, key channel (warp + 8 m) 16 + j 8 + (lane & 3) 2 + (e & 1)
+  float s[2][2][4];
 #pragma unroll
   for (int m = 0; m < 2; ++m)
 #pragma unroll
-    for (int j = 0; j < NT; ++j)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int row = (warp + 8 * m) * 16 + (lane >> 2) + half * 8, col = d0 + j * 8 + (lane & 3) * 2;
-        float2 x = make_float2(0.f, 0.f);
-        if (row < n && col < dv) x = *(const float2*)(st + (size_t)row * dv + col);
-        s[m][j][half * 2] = x.x, s[m][j][half * 2 + 1] = x.y;
+      for (int e = 0; e < 4; ++e) {
+        const int key = (warp + 8 * m) * 16 + j * 8 + (lane & 3) * 2 + (e & 1), col = d0 + (lane >> 2) + (e >> 1) * 8;
+        s[m][j][e] = key < n && col < dv ? st[(size_t)key * dv + col] : 0.f;
       }
-  auto stage_state = [&](int chunk) {    // the state before a chunk: into shared memory, and to the output kernel
-    __nv_bfloat16* out = p.before + ((size_t)chunk_slot(first, i, chunk) * p.heads + h) * 2 * n * dv + d0;
-#pragma unroll
-    for (int m = 0; m < 2; ++m) {
-      if ((warp + 8 * m) * 16 >= np) break;
-#pragma unroll
-      for (int j = 0; j < NT; ++j)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int row = (warp + 8 * m) * 16 + (lane >> 2) + half * 8, col = j * 8 + (lane & 3) * 2;
-          uint32_t hi, lo;
-          split_pair(s[m][j][half * 2], s[m][j][half * 2 + 1], hi, lo);
-          *(uint32_t*)(sh + row * VP + col) = hi;
-          *(uint32_t*)(sl + row * VP + col) = lo;
-          if (row < n && d0 + col < dv) {
-            *(uint32_t*)(out + (size_t)row * dv + col) = hi;
-            *(uint32_t*)(out + ((size_t)n + row) * dv + col) = lo;
-          }
-        }
-    }
-  };
-  stage_state(0);
   fetch(0);
-  const int m0 = (warp & 3) * 16, rows[2] = {m0 + (lane >> 2), m0 + (lane >> 2) + 8};
-  float2 u0[MINE][2];
-  float last, from[2], inv[2];           // of the chunk: c at its end and at this thread's rows, and 1 / |k|
-  auto ask = [&](int chunk) {            // for what a chunk needs in registers, one chunk ahead
-    const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
-    const float* vec = p.vec + unit * 2 * CHUNK;
-    last = vec[CHUNK - 1];
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      from[half] = vec[rows[half]];
-      inv[half] = vec[CHUNK + rows[half]];
-#pragma unroll
-      for (int j = 0; j < MINE; ++j) {
-        const int col = d0 + ((warp >> 2) + 2 * j) * 8 + (lane & 3) * 2;
-        u0[j][half] = col < dv ? *(const float2*)(p.u0 + (unit * CHUNK + rows[half]) * dv + col) : make_float2(0.f, 0.f);
-      }
-    }
-  };
-  ask(0);
+  ask();
   for (int chunk = 0; chunk < chunks; ++chunk) {
-    const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
-    const float weight[2] = {exp2f(last - from[0]) * inv[0], exp2f(last - from[1]) * inv[1]}, keep = exp2f(last);
     cp_async_wait<0>();
-    __syncthreads();                     // this chunk's operands and the state's planes are there; the chunk before is done with
+    __syncthreads();                     // this chunk's W and K are there; the chunk before is done with
     if (stages > 1 && chunk + 1 < chunks) fetch(chunk + 1);
+    const float last = next_last, keep = exp2f(last);
+    u0 = next_u0;
+    if (tid < CHUNK) weight[tid] = exp2f(last - next_c) * next_inv;
+    if (chunk + 1 < chunks) ask();
     const __nv_bfloat16* wh = ring + (stages > 1 ? chunk & 1 : 0) * stage_size;
     const __nv_bfloat16* ks = wh + (size_t)2 * CHUNK * kp;
-    float acc[MINE][3][4];
+    float acc[CHUNK / 8][4];
 #pragma unroll
-    for (int j = 0; j < MINE; ++j)
+    for (int j = 0; j < CHUNK / 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
 #pragma unroll
-      for (int x = 0; x < 3; ++x) acc[j][x][0] = acc[j][x][1] = acc[j][x][2] = acc[j][x][3] = 0.f;
-    const uint32_t w_at = smem_u32(wh + (size_t)(m0 + (mid & 1) * 8 + r) * kp + (mid >> 1) * 8), w_lo = CHUNK * kp * 2;
-#pragma unroll 4
-    for (int t = 0; t < np; t += 32) {
-      uint32_t ah[2][4], al[2][4];
+    for (int m = 0; m < 2; ++m) {
+      const int key0 = (warp + 8 * m) * 16;
+      if (key0 >= np) break;
+      uint32_t hi[4], lo[4];
 #pragma unroll
-      for (int x = 0; x < 2; ++x) {
-        ldmatrix_x4(ah[x], w_at + (t + x * 16) * 2);
-        ldmatrix_x4(al[x], w_at + w_lo + (t + x * 16) * 2);
-      }
+      for (int e = 0; e < 4; ++e) split_pair(s[m][e >> 1][(e & 1) * 2], s[m][e >> 1][(e & 1) * 2 + 1], hi[e], lo[e]);
+      const uint32_t w_at = smem_u32(wh + (size_t)((mid >> 1) * 8 + r) * kp + key0 + (mid & 1) * 8), w_lo = CHUNK * kp * 2;
+      // the three products of an accumulator stand eight others apart: none waits for the one before it
+      uint32_t w4[CHUNK / 16][4];
 #pragma unroll
-      for (int j = 0; j < MINE; ++j) {
-        uint32_t bh[4], bl[4];
-        const int at = (t + mid * 8 + r) * VP + ((warp >> 2) + 2 * j) * 8;
-        ldmatrix_x4_trans(bh, smem_u32(sh + at));
-        ldmatrix_x4_trans(bl, smem_u32(sl + at));
+      for (int j = 0; j < CHUNK / 16; ++j) ldmatrix_x4(w4[j], w_at + j * 16 * kp * 2);
 #pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          mma_16816(acc[j][0], ah[x], bh[2 * x], bh[2 * x + 1]);
-          mma_16816(acc[j][1], al[x], bh[2 * x], bh[2 * x + 1]);
-          mma_16816(acc[j][2], ah[x], bl[2 * x], bl[2 * x + 1]);
+      for (int j = 0; j < CHUNK / 8; ++j) mma_16816(acc[j], hi, w4[j >> 1][2 * (j & 1)], w4[j >> 1][2 * (j & 1) + 1]);
+#pragma unroll
+      for (int j = 0; j < CHUNK / 8; ++j) mma_16816(acc[j], lo, w4[j >> 1][2 * (j & 1)], w4[j >> 1][2 * (j & 1) + 1]);
+#pragma unroll
+      for (int j = 0; j < CHUNK / 16; ++j) ldmatrix_x4(w4[j], w_at + j * 16 * kp * 2 + w_lo);
+#pragma unroll
+      for (int j = 0; j < CHUNK / 8; ++j) mma_16816(acc[j], hi, w4[j >> 1][2 * (j & 1)], w4[j >> 1][2 * (j & 1) + 1]);
+      // the state before this chunk goes to the output kernel
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (key0 + (e >> 1) * 8 + (lane & 3) * 2 < n && d0 + (lane >> 2) + (e & 1) * 8 < dv) {
+          __nv_bfloat16* to = before_at + m * 128 + (e >> 1) * 8 + (e & 1) * 8 * n;
+          *(uint32_t*)to = hi[e];
+          *(uint32_t*)(to + lo_state) = lo[e];
         }
       }
     }
+    before_at += before_step;
+    if (warp < parts) {
+      float* to = part + ((size_t)warp * PASS_COLUMNS + (lane >> 2)) * PART_PITCH + (lane & 3) * 2;
 #pragma unroll
-    for (int j = 0; j < MINE; ++j)
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int col = ((warp >> 2) + 2 * j) * 8 + (lane & 3) * 2, e = half * 2;
-        const float a = u0[j][half].x - (acc[j][0][e] + (acc[j][1][e] + acc[j][2][e]));
-        const float c = u0[j][half].y - (acc[j][0][e + 1] + (acc[j][1][e + 1] + acc[j][2][e + 1]));
-        uint32_t hi, lo;
-        split_pair(a * weight[half], c * weight[half], hi, lo);
-        *(uint32_t*)(uh + rows[half] * VP + col) = hi;
-        *(uint32_t*)(ul + rows[half] * VP + col) = lo;
-        if (d0 + col < dv) {
-          split_pair(a, c, hi, lo);
-          __nv_bfloat16* out = p.u + (unit * 2 * CHUNK + rows[half]) * dv + d0 + col;
-          *(uint32_t*)out = hi;
-          *(uint32_t*)(out + (size_t)CHUNK * dv) = lo;
-        }
+      for (int j = 0; j < CHUNK / 8; ++j) {
+        *(float2*)(to + j * 8) = make_float2(acc[j][0], acc[j][1]);
+        *(float2*)(to + 8 * PART_PITCH + j * 8) = make_float2(acc[j][2], acc[j][3]);
       }
-    if (chunk + 1 < chunks) ask(chunk + 1);
+    }
+    __syncthreads();
+    {
+      float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+      const float* from = part + (size_t)my_col * PART_PITCH + my_row;
+#pragma unroll
+      for (int w = 0; w < PASS_WARPS; ++w) {
+        if (w >= parts) break;
+        const float4 x = *(const float4*)(from + (size_t)w * PASS_COLUMNS * PART_PITCH);
+        sum.x += x.x, sum.y += x.y, sum.z += x.z, sum.w += x.w;
+      }
+      const float4 f = *(const float4*)(weight + my_row);
+      const float u[4] = {u0.x - sum.x, u0.y - sum.y, u0.z - sum.z, u0.w - sum.w};
+      uint2 hi, lo;
+      split_pair(u[0] * f.x, u[1] * f.y, hi.x, lo.x);
+      split_pair(u[2] * f.z, u[3] * f.w, hi.y, lo.y);
+      *(uint2*)&us[0][my_col][my_row] = hi;
+      *(uint2*)&us[1][my_col][my_row] = lo;
+      if (my_valid) {
+        split_pair(u[0], u[1], hi.x, lo.x);
+        split_pair(u[2], u[3], hi.y, lo.y);
+        *(uint2*)u_at = hi;
+        *(uint2*)(u_at + lo_u) = lo;
+      }
+      u_at += u_step;
+    }
     __syncthreads();
 #pragma unroll
     for (int m = 0; m < 2; ++m) {
-      const int row0 = (warp + 8 * m) * 16;
-      if (row0 >= np) break;
+      const int key0 = (warp + 8 * m) * 16;
+      if (key0 >= np) break;
+      float more[2][4];                  // the low halves' products, a chain of their own
 #pragma unroll
-      for (int j = 0; j < NT; ++j)
+      for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[m][j][e] *= keep;
+        for (int e = 0; e < 4; ++e) s[m][j][e] *= keep, more[j][e] = 0.f;
 #pragma unroll
       for (int t = 0; t < CHUNK / 16; ++t) {
-        uint32_t a[4];
-        ldmatrix_x4_trans(a, smem_u32(ks + (size_t)(t * 16 + (mid >> 1) * 8 + r) * kp + row0 + (mid & 1) * 8));
+        uint32_t hi[4], lo[4], k4[4];
+        ldmatrix_x4(hi, smem_u32(&us[0][(mid & 1) * 8 + r][t * 16 + (mid >> 1) * 8]));
+        ldmatrix_x4(lo, smem_u32(&us[1][(mid & 1) * 8 + r][t * 16 + (mid >> 1) * 8]));
+        ldmatrix_x4_trans(k4, smem_u32(ks + (size_t)(t * 16 + (mid & 1) * 8 + r) * kp + key0 + (mid >> 1) * 8));
 #pragma unroll
-        for (int j = 0; j < NT / 2; ++j) {
-          uint32_t hi[4], lo[4];
-          const int at = (t * 16 + (mid & 1) * 8 + r) * VP + j * 16 + (mid >> 1) * 8;
-          ldmatrix_x4_trans(hi, smem_u32(uh + at));
-          ldmatrix_x4_trans(lo, smem_u32(ul + at));
-          mma_16816(s[m][2 * j], a, hi[0], hi[1]);
-          mma_16816(s[m][2 * j + 1], a, hi[2], hi[3]);
-          mma_16816(s[m][2 * j], a, lo[0], lo[1]);
-          mma_16816(s[m][2 * j + 1], a, lo[2], lo[3]);
-        }
+        for (int j = 0; j < 2; ++j) mma_16816(s[m][j], hi, k4[2 * j], k4[2 * j + 1]);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) mma_16816(more[j], lo, k4[2 * j], k4[2 * j + 1]);
       }
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[m][j][e] += more[j][e];
     }
-    if (chunk + 1 < chunks) stage_state(chunk + 1);      // its readers are behind the barrier above
     if (stages == 1 && chunk + 1 < chunks) {
       __syncthreads();                   // K is used up
       fetch(chunk + 1);
@@ -792,21 +803,21 @@ __global__ void __launch_bounds__(PASS_THREADS) delta_pass_kernel(const Delta p,
 #pragma unroll
   for (int m = 0; m < 2; ++m)
 #pragma unroll
-    for (int j = 0; j < NT; ++j)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int row = (warp + 8 * m) * 16 + (lane >> 2) + half * 8, col = d0 + j * 8 + (lane & 3) * 2;
-        if (row < n && col < dv) *(float2*)(st + (size_t)row * dv + col) = make_float2(s[m][j][half * 2], s[m][j][half * 2 + 1]);
+      for (int e = 0; e < 4; ++e) {
+        const int key = (warp + 8 * m) * 16 + j * 8 + (lane & 3) * 2 + (e & 1), col = d0 + (lane >> 2) + (e >> 1) * 8;
+        if (key < n && col < dv) st[(size_t)key * dv + col] = s[m][j][e];
       }
 }
 
 // ---------------------------------------------------------------------------------------
 // chunked: output
 // ---------------------------------------------------------------------------------------
-constexpr int OUT_THREADS = 256, OUT_DVT = 64, OUT_VP = OUT_DVT + 8;
+constexpr int OUT_THREADS = 256, OUT_DVT = 64;
 __host__ __device__ inline size_t output_smem(int n) {
   const int np = (n + 15) & ~15;
-  return 2 * ((size_t)2 * CHUNK * (np + 8) + (size_t)2 * (np + CHUNK) * OUT_VP);
+  return 2 * ((size_t)2 * (CHUNK + OUT_DVT) * (np + 8) + (size_t)2 * OUT_DVT * U_PITCH);
 }
 
 // A chunk's read-outs, 64 value columns a block: a warp 16 tokens x 32 columns.
@@ -826,20 +837,20 @@ __global__ void __launch_bounds__(OUT_THREADS) delta_output_kernel(const Delta p
   const size_t unit = (size_t)chunk_slot(first, i, chunk) * p.heads + h;
   __nv_bfloat16* qs = (__nv_bfloat16*)raw;                // [CHUNK][kp]
   __nv_bfloat16* ks = qs + (size_t)CHUNK * kp;
-  __nv_bfloat16* sh = ks + (size_t)CHUNK * kp;            // [np][OUT_VP]
-  __nv_bfloat16* sl = sh + (size_t)np * OUT_VP;
-  __nv_bfloat16* uh = sl + (size_t)np * OUT_VP;           // [CHUNK][OUT_VP]
-  __nv_bfloat16* ul = uh + (size_t)CHUNK * OUT_VP;
+  __nv_bfloat16* sh = ks + (size_t)CHUNK * kp;            // [OUT_DVT][kp]
+  __nv_bfloat16* sl = sh + (size_t)OUT_DVT * kp;
+  __nv_bfloat16* uh = sl + (size_t)OUT_DVT * kp;          // [OUT_DVT][U_PITCH]
+  __nv_bfloat16* ul = uh + (size_t)OUT_DVT * U_PITCH;
   const int valid = min(OUT_DVT, dv - d0);
   fetch_rows(qs, kp, (const __nv_bfloat16*)p.q + token0 * p.q_ld + g * n, p.q_ld, CHUNK, count, np, n);
   fetch_rows(ks, kp, (const __nv_bfloat16*)p.k + token0 * p.k_ld + g * n, p.k_ld, CHUNK, count, np, n);
-  const __nv_bfloat16* before = p.before + unit * 2 * n * dv + d0;
-  fetch_rows(sh, OUT_VP, before, dv, np, n, OUT_DVT, valid);
-  fetch_rows(sl, OUT_VP, before + (size_t)n * dv, dv, np, n, OUT_DVT, valid);
+  const __nv_bfloat16* before = p.before + (unit * 2 * dv + d0) * n;
+  fetch_rows(sh, kp, before, n, OUT_DVT, valid, np, n);
+  fetch_rows(sl, kp, before + (size_t)dv * n, n, OUT_DVT, valid, np, n);
   cp_async_commit();
-  const __nv_bfloat16* u = p.u + unit * 2 * CHUNK * dv + d0;
-  fetch_rows(uh, OUT_VP, u, dv, CHUNK, CHUNK, OUT_DVT, valid);
-  fetch_rows(ul, OUT_VP, u + (size_t)CHUNK * dv, dv, CHUNK, CHUNK, OUT_DVT, valid);
+  const __nv_bfloat16* u = p.u + (unit * 2 * dv + d0) * CHUNK;
+  fetch_rows(uh, U_PITCH, u, CHUNK, OUT_DVT, valid, CHUNK, CHUNK);
+  fetch_rows(ul, U_PITCH, u + (size_t)dv * CHUNK, CHUNK, OUT_DVT, valid, CHUNK, CHUNK);
   cp_async_commit();
   if (tid < CHUNK) {
     cumulative[tid] = p.vec[unit * 2 * CHUNK + tid];
@@ -847,14 +858,9 @@ __global__ void __launch_bounds__(OUT_THREADS) delta_output_kernel(const Delta p
   }
   cp_async_wait<1>();
   __syncthreads();
-  for (int t = warp; t < CHUNK; t += OUT_THREADS / 32) {
-    float qq = 0.f;
-    for (int e = lane; e < np; e += 32) {
-      const float q = __bfloat162float(qs[t * kp + e]);
-      qq = fmaf(q, q, qq);
-    }
-    qq = all_sum(qq);
-    if (lane == 0) q_inv[t] = inverse_root(qq + p.key_eps) * p.q_scale;
+  {
+    const float qq = row_squares(qs, kp, np, tid >> 2);
+    if ((tid & 3) == 0) q_inv[tid >> 2] = inverse_root(qq + p.key_eps) * p.q_scale;
   }
   const int tile = warp & 3, row0 = tile * 16, col0 = (warp >> 2) * 32;
   float acc[4][4];
@@ -867,11 +873,11 @@ __global__ void __launch_bounds__(OUT_THREADS) delta_output_kernel(const Delta p
     ldmatrix_x4(a, q_at + t * 32);
 #pragma unroll
     for (int plane = 0; plane < 2; ++plane) {
-      const __nv_bfloat16* from = (plane == 0 ? sh : sl) + (t * 16 + (mid & 1) * 8 + r) * OUT_VP + col0 + (mid >> 1) * 8;
+      const __nv_bfloat16* from = (plane == 0 ? sh : sl) + (size_t)(col0 + (mid >> 1) * 8 + r) * kp + t * 16 + (mid & 1) * 8;
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         uint32_t s4[4];
-        ldmatrix_x4_trans(s4, smem_u32(from + j * 16));
+        ldmatrix_x4(s4, smem_u32(from + (size_t)j * 16 * kp));
         mma_16816(acc[2 * j], a, s4[0], s4[1]);
         mma_16816(acc[2 * j + 1], a, s4[2], s4[3]);
       }
@@ -901,28 +907,33 @@ __global__ void __launch_bounds__(OUT_THREADS) delta_output_kernel(const Delta p
       mma_16816(s[1], a, k4[2], k4[3]);
     }
 #pragma unroll
-    for (int w = 0; w < 2; ++w)
+    for (int w = 0; w < 2; ++w) {
+      const int token = t * 16 + w * 8 + (lane & 3) * 2;
+      const float2 c2 = *(const float2*)(cumulative + token), i2 = *(const float2*)(k_inv + token);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int token = t * 16 + w * 8 + (lane & 3) * 2 + (e & 1), half = e >> 1;
-        s[w][e] = token <= rows[half] ? s[w][e] * (scale[half] * k_inv[token] * fast_exp2(at_row[half] - cumulative[token])) : 0.f;
+        const int half = e >> 1;
+        const float f = scale[half] * (e & 1 ? i2.y : i2.x) * fast_exp2(at_row[half] - (e & 1 ? c2.y : c2.x));
+        s[w][e] = token + (e & 1) <= rows[half] ? s[w][e] * f : 0.f;
       }
+    }
     uint32_t hi[4], lo[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) split_pair(s[e >> 1][(e & 1) * 2], s[e >> 1][(e & 1) * 2 + 1], hi[e], lo[e]);
+    uint32_t u4[2][4], l4[2][4];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
-      uint32_t u4[4], l4[4];
-      const int at = (t * 16 + (mid & 1) * 8 + r) * OUT_VP + col0 + j * 16 + (mid >> 1) * 8;
-      ldmatrix_x4_trans(u4, smem_u32(uh + at));
-      ldmatrix_x4_trans(l4, smem_u32(ul + at));
-      mma_16816(acc[2 * j], hi, u4[0], u4[1]);
-      mma_16816(acc[2 * j + 1], hi, u4[2], u4[3]);
-      mma_16816(acc[2 * j], lo, u4[0], u4[1]);
-      mma_16816(acc[2 * j + 1], lo, u4[2], u4[3]);
-      mma_16816(acc[2 * j], hi, l4[0], l4[1]);
-      mma_16816(acc[2 * j + 1], hi, l4[2], l4[3]);
+      const int at = (col0 + j * 16 + (mid >> 1) * 8 + r) * U_PITCH + t * 16 + (mid & 1) * 8;
+      ldmatrix_x4(u4[j], smem_u32(uh + at));
+      ldmatrix_x4(l4[j], smem_u32(ul + at));
     }
+#pragma unroll
+    for (int x = 0; x < 3; ++x)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const uint32_t* from = x == 2 ? l4[j >> 1] : u4[j >> 1];
+        mma_16816(acc[j], x == 1 ? lo : hi, from[2 * (j & 1)], from[2 * (j & 1) + 1]);
+      }
   }
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -958,11 +969,13 @@ Delta delta_of(float* o, float* state, long long slot_stride, const void* q, int
   return p;
 }
 
-template <int DVT>
 int launch_pass(const Delta& p, int listed, cudaStream_t s) {
-  const int stages = pass_smem(p.n, DVT, 2) <= SMEM_MOST ? 2 : 1;
-  if (int err = allow_smem(delta_pass_kernel<DVT>, SMEM_MOST, "gated_delta_chunked")) return err;
-  launch_kernel(delta_pass_kernel<DVT>, dim3((p.dv + DVT - 1) / DVT, p.heads, listed), PASS_THREADS, pass_smem(p.n, DVT, stages), s, p, stages);
+  // Two stages of W and K while every block has an SM to itself; one when there are more blocks, which then share SMs.
+  const dim3 grid((p.dv + PASS_COLUMNS - 1) / PASS_COLUMNS, p.heads, listed);
+  const bool alone = (long long)grid.x * grid.y * grid.z <= 148;
+  const int stages = alone && pass_smem(p.n, 2) <= SMEM_MOST ? 2 : 1;
+  if (int err = allow_smem(delta_pass_kernel, SMEM_MOST, "gated_delta_chunked")) return err;
+  launch_kernel(delta_pass_kernel, grid, PASS_THREADS, pass_smem(p.n, stages), s, p, stages);
   return check_launch("gated_delta_pass");
 }
 
@@ -1012,7 +1025,7 @@ PAE_EXPORT int pae_gated_delta_pitch(int n) { return pitch_of(n); }
 
 // The entries that bring more than one token, bfloat16. list: `listed` entries to look at (null: all, and
 // those of one token are passed over). Scratch for tokens / 64 + listed chunks, per chunk and head: wk bfloat16
-// [3, 64, pitch], u0 floats [64, dv], u bfloat16 [2, 64, dv], before bfloat16 [2, n, dv], vec floats [2, 64]. Three launches.
+// [3, 64, pitch], u0 floats [dv, 64], u bfloat16 [2, dv, 64], before bfloat16 [2, dv, n], vec floats [2, 64]. Three launches.
 PAE_EXPORT int pae_gated_delta_chunked(float* o, float* state, long long slot_stride, const void* q, int q_ld, const void* k, int k_ld,
                                        const void* v, int v_ld, const float* log_decay, const float* beta, float key_eps, float q_scale,
                                        const int* q_start, const int* state_slot, const int* list, int listed, int max_q_len, int heads,
@@ -1031,9 +1044,7 @@ PAE_EXPORT int pae_gated_delta_chunked(float* o, float* state, long long slot_st
   if (int err = allow_smem(delta_solve_kernel, SMEM_MOST, "gated_delta_chunked")) return err;
   launch_kernel(delta_solve_kernel, dim3(chunks, heads, listed), SOLVE_THREADS, solve_smem(n, dv), s, p);
   if (int err = check_launch("gated_delta_solve")) return err;
-  // wider blocks read W and K fewer times; narrow ones keep the SMs busy while the heads are few
-  const bool wide = (long long)listed * heads * ((dv + 31) / 32) >= 148;
-  if (int err = wide ? launch_pass<32>(p, listed, s) : launch_pass<16>(p, listed, s)) return err;
+  if (int err = launch_pass(p, listed, s)) return err;
   if (int err = allow_smem(delta_output_kernel, SMEM_MOST, "gated_delta_chunked")) return err;
   launch_kernel(delta_output_kernel, dim3(chunks * ((dv + OUT_DVT - 1) / OUT_DVT), heads, listed), OUT_THREADS, output_smem(n), s, p);
   return check_launch("gated_delta_output");

@@ -331,6 +331,15 @@ __global__ void __launch_bounds__(PER <= 4 ? 512 : 256) post_norm_row_kernel(con
   }
 }
 
+// The stream rounded, nothing else: the first sublayer's read.
+__global__ void __launch_bounds__(256) round_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ x, long long total) {
+  dependent_launch_prologue();
+  const long long at = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (at >= total) return;
+  put<4>(out + at, get<4>(x + at));
+  if (at + 4 < total) put<4>(out + at + 4, get<4>(x + at + 4));
+}
+
 template <typename TO, int BRANCHES>
 int launch_row(const PostNorm& p, int rows, cudaStream_t s) {
   const int pieces = p.width / 4;
@@ -383,6 +392,10 @@ PAE_EXPORT int pae_post_norm(float* x_new, void* read, const float* x, int branc
   for (int b = 0; b < MAX_BRANCHES; ++b) {
     if (b < branches && (p.y[b] == nullptr || p.planes[b] < 1)) return fail(2, "post_norm: branch %d has %d planes", b, p.planes[b]);
     wide = wide && aligned16(p.y[b]) && aligned16(p.w[b]);
+  }
+  if (wide && branches == 0 && read_w == nullptr && x_new == nullptr && read_dtype == kBF16) {
+    launch_kernel(round_kernel, (unsigned)((p.total / 4 + 511) / 512), 256, 0, (cudaStream_t)stream, (__nv_bfloat16*)read, x, p.total);
+    return check_launch("post_norm_round");
   }
   if (wide && width <= 8192 && (branches == 1 || branches == 2)) {
     cudaStream_t s = (cudaStream_t)stream;
