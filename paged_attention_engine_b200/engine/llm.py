@@ -112,11 +112,12 @@ class Engine:
             if own is not None:
                 extra += int(own(num_tokens))
                 return
-            for value in vars(obj).values():
-                if isinstance(value, torch.Tensor):
-                    seen[value.data_ptr()] = value.numel() * value.element_size()
-                elif hasattr(value, "runtime") and value is not obj:
-                    visit(value)
+            for held in vars(obj).values():
+                for value in held if isinstance(held, (list, tuple)) else (held,):
+                    if isinstance(value, torch.Tensor):
+                        seen[value.data_ptr()] = value.numel() * value.element_size()
+                    elif hasattr(value, "runtime") and value is not obj:
+                        visit(value)
 
         for part in self.model.parts():
             visit(part)
